@@ -98,6 +98,36 @@ def _build(sources: list[Path], headers: list[Path], out: Path, compiler: list[s
     return True
 
 
+# The kernels a layer-stack model is served with (serve.stack): enough for a checkout that only serves, in a
+# fraction of the time the whole library takes.
+SERVE_SOURCES = ("elementwise", "flash_fwd", "gemm_f32", "gemm_tcgen05", "host_common", "latent_attn_tc", "latent_kv", "moe",
+                 "kv_attn_tc", "residual_stream", "serving")
+
+
+def build_serving_kernels(verbose: bool = False) -> Path:
+    """``libcogito_kernels_serve.so``: the subset of the kernel library in SERVE_SOURCES."""
+    srcs = [ROOT / "csrc" / "kernels" / f"{name}.cu" for name in SERVE_SOURCES]
+    out = LIB_DIR / "libcogito_kernels_serve.so"
+    nvcc = _nvcc()
+    _build(srcs, _kernel_headers(), out, [nvcc] + NVCC_FLAGS + ["-I", str(ROOT / "include")],
+           [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC", "-cudart", "shared"], "kernels", verbose)
+    return out
+
+
+def ensure_serving(verbose: bool = False) -> Path:
+    """The kernel library to serve from: the whole one if it has been built, else the serving subset (built now
+    if it is missing)."""
+    full, part = LIB_DIR / "libcogito_kernels.so", LIB_DIR / "libcogito_kernels_serve.so"
+    if full.exists():
+        return full
+    return part if part.exists() else build_serving_kernels(verbose)
+
+
+def _kernel_headers() -> list[Path]:
+    return (list((ROOT / "csrc").rglob("*.cuh")) + list((ROOT / "csrc").rglob("*.h")) + list((ROOT / "csrc").rglob("*.inc"))
+            + list((ROOT / "include").glob("*.h")))
+
+
 def build_kernels(verbose: bool = False, debug_bounds: bool = False) -> Path:
     """debug_bounds: the same sources with -DCGK_DEBUG_BOUNDS as ``libcogito_kernels_dbg.so``: indices
     that come from data or from tile edges are checked, the first violation per source file is
@@ -105,8 +135,7 @@ def build_kernels(verbose: bool = False, debug_bounds: bool = False) -> Path:
     makes the package load that library, and ``ops._lib.assert_device_ok`` (which the GPU tests
     call after every test) then fails on a recorded violation."""
     srcs = sorted((ROOT / "csrc" / "kernels").glob("*.cu")) + sorted((ROOT / "csrc" / "comm").glob("*.cu"))
-    hdrs = (list((ROOT / "csrc").rglob("*.cuh")) + list((ROOT / "csrc").rglob("*.h")) + list((ROOT / "csrc").rglob("*.inc"))
-            + list((ROOT / "include").glob("*.h")))
+    hdrs = _kernel_headers()
     out = LIB_DIR / ("libcogito_kernels_dbg.so" if debug_bounds else "libcogito_kernels.so")
     nvcc = _nvcc()
     flags = NVCC_FLAGS + (["-DCGK_DEBUG_BOUNDS"] if debug_bounds else [])
@@ -165,6 +194,7 @@ def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__)
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--capi", action="store_true")
+    ap.add_argument("--serving", action="store_true", help="only build libcogito_kernels_serve.so, the kernels layer-stack models are served with")
     ap.add_argument("--sanitize", action="store_true", help="only build the ASan + UBSan copy of the host runtime")
     ap.add_argument("--debug-bounds", action="store_true",
                     help="only build libcogito_kernels_dbg.so: every kernel with index checks that record the first violation")
@@ -175,6 +205,9 @@ def main() -> None:
         return
     if args.debug_bounds:
         print(build_kernels(args.verbose, debug_bounds=True))
+        return
+    if args.serving:
+        print(build_serving_kernels(args.verbose))
         return
     if args.kernels or not args.capi:
         print(build_kernels(args.verbose))

@@ -15,10 +15,14 @@ import torch
 
 # COGITO_KERNELS_DEBUG=1 selects the index-checking build (python -m cogito_b200.build --debug-bounds)
 _DEBUG = os.environ.get("COGITO_KERNELS_DEBUG", "0") not in ("", "0")
-_LIB_PATH = Path(__file__).resolve().parent.parent / "lib" / ("libcogito_kernels_dbg.so" if _DEBUG else "libcogito_kernels.so")
+_LIB_DIR = Path(__file__).resolve().parent.parent / "lib"
+_LIB_PATH = _LIB_DIR / ("libcogito_kernels_dbg.so" if _DEBUG else "libcogito_kernels.so")
+if not _DEBUG and not _LIB_PATH.exists() and (_LIB_DIR / "libcogito_kernels_serve.so").exists():
+    _LIB_PATH = _LIB_DIR / "libcogito_kernels_serve.so"           # a checkout that only serves: part of the kernels
 _lib = None
 # source files that carry index checks in the debug build (one recorded violation each)
-_BOUNDS_FILES = ("gemm_tcgen05", "softmax_ce", "serving", "elementwise", "flash_fwd", "flash_bwd")
+_BOUNDS_FILES = ("gemm_tcgen05", "softmax_ce", "serving", "elementwise", "flash_fwd", "flash_bwd", "residual_stream", "latent_kv",
+                 "latent_attn_tc", "moe")
 
 
 class KernelError(RuntimeError):
@@ -100,6 +104,20 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_sample": [vp, i, ll, i, i, f, i, f, c_ulonglong, vp, vp, vp, vp],
         "cgk_spec_accept": [vp, vp, vp, i, i, i, c_ulonglong, vp, vp, vp, vp, vp, vp],
         "cgk_tree_mask": [vp, i, i, vp, vp, vp],
+        "cgk_embed_sinusoid": [vp, vp, vp, i, f, vp, vp, vp, i, i, i, i, vp],
+        "cgk_stream_update": [vp, vp],
+        "cgk_rms_rows": [vp, vp, i, i, vp, vp, i, i, f, vp],
+        "cgk_gemm_f32": [vp, vp, vp, i, i, i, i, ll, ll, ll, ll, ll, ll, i, vp],
+        "cgk_latent_norm_append": [vp, vp, i, ll, vp, vp, i, f, vp, vp, i, vp],
+        "cgk_latent_gather": [vp, i, i, vp, vp],
+        "cgk_latent_attention": [vp, vp, vp, i, i, vp, i, vp],
+        "cgk_latent_attention_tc_ok": [i, i, i],
+        "cgk_moe_route": [vp, vp, i, i, i, i, i, i, vp, vp, vp, vp, vp],
+        "cgk_moe_plan": [vp, i, vp, vp, vp, i, vp],
+        "cgk_moe_gather": [vp, vp, i, i, i, vp, vp, vp, i, i, vp],
+        "cgk_gemm_grouped_bf16": [POINTER(GemmArgs), vp, vp, vp],
+        "cgk_swiglu_tiles": [vp, vp, vp, i, i, vp],
+        "cgk_expert_rows": [i, vp, vp, i, i, i, vp, vp, vp, vp, i, i, vp],
     }
     for name, argtypes in sigs.items():
         fn = getattr(L, name, None)
@@ -113,13 +131,17 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_int4_tiles_bytes": [i, i],
         "cgk_int4_wa_tiles_bytes": [i, i],
         "cgk_int4_gemm_counters": [i, i],
+        "cgk_latent_attention_scratch_floats": [i, i, i, i],
     }.items():
-        fn = getattr(L, name)
+        fn = getattr(L, name, None)
+        if fn is None:                              # a library built from part of the sources
+            continue
         fn.argtypes = argtypes
         fn.restype = c_longlong
-    L.cgk_grad_stats_scratch_elems.argtypes = [ll]
-    L.cgk_reduce_all_scratch_elems.argtypes = [ll]
-    L.cgk_scaler_state_bytes.argtypes = []
+    for name, argtypes in {"cgk_grad_stats_scratch_elems": [ll], "cgk_reduce_all_scratch_elems": [ll], "cgk_scaler_state_bytes": []}.items():
+        fn = getattr(L, name, None)
+        if fn is not None:
+            fn.argtypes = argtypes
 
 
 def available() -> bool:

@@ -104,16 +104,19 @@ def _fill_common(a: FlashArgs, q, k, v, o, lse, scale, causal, window, alibi):
     a.alibi_slopes = alibi.data_ptr() if alibi is not None else None
 
 
-def flash_forward(q, k, v, *, causal=False, window=-1, scale=None, alibi=None):
-    """Returns (o [B,Tq,Hq,D] bf16, lse [B,Hq,Tq] fp32).  q/k/v may be strided views."""
+def flash_forward(q, k, v, *, causal=False, window=-1, scale=None, alibi=None, out=None):
+    """Returns (o [B,Tq,Hq,D] bf16, lse [B,Hq,Tq] fp32).  q/k/v may be strided views; ``out`` (same shape as q,
+    may be a strided view) receives o."""
     B, Tq, Hq, D = q.shape
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     if not q.is_cuda:
         o, lse = attention_reference(q, k, v, causal=causal, window=window, scale=scale, alibi=alibi)
+        if out is not None:
+            return out.copy_(o), lse
         return o.to(q.dtype), lse
     if q.dtype != torch.bfloat16:
         raise TypeError("flash_forward: CUDA tensors must be bf16")
-    o = torch.empty(B, Tq, Hq, D, device=q.device, dtype=torch.bfloat16)
+    o = torch.empty(B, Tq, Hq, D, device=q.device, dtype=torch.bfloat16) if out is None else out
     lse = torch.empty(B, Hq, Tq, device=q.device, dtype=torch.float32)
     a = FlashArgs()
     _fill_common(a, q, k, v, o, lse, scale, causal, window, alibi)

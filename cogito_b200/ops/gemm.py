@@ -4,7 +4,7 @@
 where each operand may be stored K-major or MN-major (see
 ``include/cogito_kernels.h``).  CUDA tensors run ``cgk_gemm_bf16``; CPU tensors
 run an fp32 restatement of the same formula, which is also the oracle of the GPU
-tests.
+tests.  Two fp32 CUDA operands run a plain product in true fp32 (``cgk_gemm_f32``).
 """
 from __future__ import annotations
 
@@ -108,6 +108,20 @@ def _ld(t: torch.Tensor) -> int:
     return t.stride(-2) if t.shape[-2] > 1 else max(t.shape[-1], t.stride(-2))
 
 
+def _gemm_f32(a, b, b_mn, out, batch_shape, batch, M, N, K):
+    """True fp32 on the CUDA cores (models served in fp32); no tensor-core mode is involved."""
+    if out is None:
+        out = torch.empty(*batch_shape, M, N, device=a.device, dtype=torch.float32)
+    elif out.shape[-2:] != (M, N) or out.dtype != torch.float32 or out.stride(-1) != 1:
+        raise ValueError("gemm: fp32 operands need a row-major fp32 output of the product's shape")
+    a3, b3, o3 = (t.reshape(batch, *t.shape[-2:]) if t.dim() != 3 else t for t in (a, b, out))
+    a3, b3 = (t if t.stride(-1) == 1 else t.contiguous() for t in (a3, b3))
+    _lib.check(_lib.lib().cgk_gemm_f32(a3.data_ptr(), b3.data_ptr(), o3.data_ptr(), M, N, K, batch, _ld(a3), _ld(b3), _ld(o3), a3.stride(0),
+                                       b3.stride(0), o3.stride(0), int(b_mn), _lib.stream_ptr()), "cgk_gemm_f32")
+    _lib.count_launch()
+    return out
+
+
 def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = False,
          out: torch.Tensor | None = None, out_dtype: torch.dtype = torch.bfloat16,
          bias: torch.Tensor | None = None, act: str | None = None,
@@ -156,8 +170,13 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
             return out
         return ref
 
+    if a.dtype == torch.float32 and b.dtype == torch.float32:
+        if a_mn or bias is not None or act not in (None, "none") or residual is not None or aux_out is not None or aux_in is not None \
+                or accumulate or alpha != 1.0 or rope is not None:
+            raise TypeError("gemm: fp32 CUDA operands take plain products only (the epilogues are bf16)")
+        return _gemm_f32(a, b, b_mn, out, batch_shape, batch, M, N, K)
     if a.dtype != torch.bfloat16 or b.dtype != torch.bfloat16:
-        raise TypeError("gemm: CUDA operands must be bf16")
+        raise TypeError("gemm: CUDA operands must both be bf16 (or both fp32)")
     if a.stride(-1) != 1:
         a = a.contiguous()
     if b.stride(-1) != 1:

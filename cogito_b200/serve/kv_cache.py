@@ -1,18 +1,23 @@
-"""Paged INT4 key/value cache and attention over it.
+"""Paged caches of the serving engines and attention over them: INT4 keys / values, and latents.
 
-Per layer the pool is ``pages[num_pages, page_size, heads, D/2]`` bytes plus fp32 scales
+``PagedCache`` holds what both share: the page table, sequence slots and lengths.
+
+INT4 (``PagedKVCacheInt4``): per layer the pool is ``pages[num_pages, page_size, heads, D/2]`` bytes plus fp32 scales
 ``[num_pages, page_size, heads, D/group]`` (one token's bytes equal the reference layout
 ``[layers, max_seq, heads, head_dim/2]`` of cg_kv_cache_int4, src/quantize/int4.c:116-145; a
 single page of ``max_seq`` tokens reproduces it exactly).  ``lengths`` counts committed tokens
 per sequence once, whatever the number of layers (the reference advances it on every
 append, src/quantize/int4.c:233).  Rejected speculative tokens are dropped by not advancing
 ``lengths`` past them.
+
+Latents (``PagedLatentCache``): per layer ``pages[num_pages, page_size, rank]`` in bf16 or fp32, one short row
+per token from which every head's key and value follow (csrc/kernels/latent_kv.cu, latent_attn_tc.cu).
 """
 from __future__ import annotations
 
 import ctypes
 import math
-from ctypes import Structure, c_int32, c_void_p
+from ctypes import Structure, c_float, c_int32, c_void_p
 
 import torch
 
@@ -27,36 +32,94 @@ class KvArgs(Structure):
                 ("page_size", c_int32), ("max_pages", c_int32)]
 
 
-class PagedKVCacheInt4:
+class PagedCache:
+    """Page table, sequence slots and committed lengths, whatever a page holds.
+
+    ``n_pages=None``: identity placement, slot b owns pages b * max_pages .. (a fixed batch of sequences; any
+    permutation of ``page_table`` works).  Otherwise the pool has ``n_pages`` pages and a sequence takes them as
+    it grows: ``open`` a slot, ``reserve`` room before a step, ``close`` it and its pages serve other sequences."""
+
+    def __init__(self, batch: int, max_seq_len: int, page_size: int, device="cpu", n_pages: int | None = None):
+        self.batch, self.page_size = batch, page_size
+        self.max_pages = (max_seq_len + page_size - 1) // page_size
+        self.device = torch.device(device)
+        self.pooled = n_pages is not None
+        self.n_pages = n_pages if self.pooled else batch * self.max_pages
+        self.lengths = torch.zeros(batch, dtype=torch.int32, device=self.device)
+        if self.pooled:
+            self.page_table = torch.zeros(batch, self.max_pages, dtype=torch.int32, device=self.device)
+            self._free_pages = list(range(self.n_pages - 1, -1, -1))
+            self._free_slots = list(range(batch - 1, -1, -1))
+            self._owned: dict[int, list[int]] = {}
+        else:
+            self.page_table = torch.arange(self.n_pages, dtype=torch.int32, device=self.device).view(batch, self.max_pages)
+
+    def reset(self):
+        self.lengths.zero_()
+        if self.pooled:
+            for slot in list(self._owned):
+                self.close(slot)
+
+    def commit(self, n_tokens):
+        """Advance the lengths (int or per-sequence tensor) after the appended tokens are accepted."""
+        self.lengths += n_tokens
+
+    # ------------------------------------------------------- slots and pages of a pooled cache
+    def open(self) -> int:
+        """Takes a free sequence slot."""
+        if not self._free_slots:
+            raise RuntimeError("no free sequence slot")
+        slot = self._free_slots.pop()
+        self._owned[slot] = []
+        return slot
+
+    def free_slots(self) -> int:
+        return len(self._free_slots)
+
+    def free_pages(self) -> int:
+        return len(self._free_pages)
+
+    def pages_for(self, length: int) -> int:
+        return (length + self.page_size - 1) // self.page_size
+
+    def reserve(self, slot: int, length: int):
+        """Gives the sequence in ``slot`` the pages that ``length`` tokens need."""
+        own = self._owned[slot]
+        need = self.pages_for(length)
+        if need <= len(own):
+            return
+        if need > self.max_pages:
+            raise ValueError(f"a sequence of {length} tokens exceeds the cache's {self.max_pages * self.page_size}")
+        if need - len(own) > len(self._free_pages):
+            raise RuntimeError(f"the page pool is exhausted: {need - len(own)} pages wanted, {len(self._free_pages)} free")
+        first = len(own)
+        own.extend(self._free_pages.pop() for _ in range(need - first))
+        self.page_table[slot, first:need] = torch.tensor(own[first:], dtype=torch.int32).to(self.device)
+
+    def close(self, slot: int):
+        """Returns the slot and its pages."""
+        self._free_pages.extend(reversed(self._owned.pop(slot)))
+        self._free_slots.append(slot)
+
+
+class PagedKVCacheInt4(PagedCache):
     def __init__(self, num_layers: int, batch: int, max_seq_len: int, heads: int, head_dim: int, group: int = 32,
                  page_size: int = 64, device="cpu"):
         if head_dim % group or group % 8:
             raise ValueError("group must be a multiple of 8 that divides head_dim")
-        self.num_layers, self.batch, self.heads, self.D, self.group = num_layers, batch, heads, head_dim, group
-        self.page_size = page_size
-        self.max_pages = (max_seq_len + page_size - 1) // page_size
-        self.device = torch.device(device)
-        n_pages = batch * self.max_pages
+        super().__init__(batch, max_seq_len, page_size, device)
+        self.num_layers, self.heads, self.D, self.group = num_layers, heads, head_dim, group
+        n_pages = self.n_pages
         G = head_dim // group
         mk = lambda *s, dt: torch.zeros(*s, dtype=dt, device=self.device)
         self.k_pages = [mk(n_pages, page_size, heads, head_dim // 2, dt=torch.uint8) for _ in range(num_layers)]
         self.v_pages = [mk(n_pages, page_size, heads, head_dim // 2, dt=torch.uint8) for _ in range(num_layers)]
         self.k_scales = [mk(n_pages, page_size, heads, G, dt=torch.float32) for _ in range(num_layers)]
         self.v_scales = [mk(n_pages, page_size, heads, G, dt=torch.float32) for _ in range(num_layers)]
-        # identity placement: sequence b owns pages b*max_pages .. ; any permutation works
-        self.page_table = torch.arange(n_pages, dtype=torch.int32, device=self.device).view(batch, self.max_pages)
-        self.lengths = torch.zeros(batch, dtype=torch.int32, device=self.device)
         self._scratch = None
 
     def nbytes(self) -> int:
         return sum(t.numel() * t.element_size() for ts in (self.k_pages, self.v_pages, self.k_scales, self.v_scales) for t in ts)
-
-    def reset(self):
-        self.lengths.zero_()
-
-    def commit(self, n_tokens):
-        """Advance the lengths (int or per-sequence tensor) after the appended tokens are accepted."""
-        self.lengths += n_tokens
 
     def _args(self, layer: int) -> KvArgs:
         a = KvArgs()
@@ -138,4 +201,97 @@ class PagedKVCacheInt4:
             mask = torch.arange(n)[None, :] > (torch.arange(Tq)[:, None] + n - Tq)
             s = s.masked_fill(mask[None], float("-inf"))
             out[b] = torch.einsum("hqk,khd->qhd", torch.softmax(s, -1), v).to(q.dtype)
+        return out
+
+
+class LatentArgs(Structure):
+    """Mirror of ``cgk_latent_args`` (include/cogito_kernels.h)."""
+
+    _fields_ = [("pages", c_void_p), ("page_table", c_void_p), ("slot", c_void_p), ("pos", c_void_p),
+                ("R", c_int32), ("page_size", c_int32), ("max_pages", c_int32), ("slots", c_int32), ("n_pages", c_int32),
+                ("heads", c_int32), ("fp32", c_int32), ("scale", c_float)]
+
+
+class PagedLatentCache(PagedCache):
+    """``ranks``: latent size of every layer run (layers may differ).  Pages start as zeros and only ever receive
+    finite rows: the tensor-core kernel reads whole pages and gives keys beyond the sequence the weight 0."""
+
+    def __init__(self, ranks, batch: int, max_seq_len: int, page_size: int = 64, device="cpu", dtype=torch.bfloat16, n_pages: int | None = None):
+        super().__init__(batch, max_seq_len, page_size, device, n_pages)
+        self.ranks, self.dtype = list(ranks), dtype
+        self.pages = [torch.zeros(self.n_pages, page_size, r, dtype=dtype, device=self.device) for r in self.ranks]
+
+    def nbytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in self.pages)
+
+    def _args(self, layer: int, slot=None, pos=None, heads: int = 0, scale: float = 1.0) -> LatentArgs:
+        a = LatentArgs()
+        a.pages, a.page_table = self.pages[layer].data_ptr(), self.page_table.data_ptr()
+        # the struct's users check for null; the gather does not look at slot and pos
+        a.slot, a.pos = _lib.ptr(slot), _lib.ptr(pos)
+        a.R, a.page_size, a.max_pages, a.slots, a.n_pages = self.ranks[layer], self.page_size, self.max_pages, self.batch, self.n_pages
+        a.heads, a.fp32, a.scale = heads, int(self.dtype == torch.float32), float(scale)
+        return a
+
+    def _place(self, slot, pos):
+        page = self.page_table[slot.long(), (pos // self.page_size).long()].long()
+        return page, (pos % self.page_size).long()
+
+    def norm_append(self, layer: int, lat, wq, wc, eps: float, slot, pos, keep: bool):
+        """lat [N, q_rank + rank] (the two down-projections side by side) -> the RMS-normed query latents [N, q_rank];
+        the RMS-normed key/value latents go to their cache places (and come back as well with ``keep``)."""
+        qr, R, N = wq.shape[0], self.ranks[layer], lat.shape[0]
+        if not lat.is_cuda:
+            def norm(v, w):
+                v = v.float()
+                return (v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps) * w).to(self.dtype)
+            c = norm(lat[:, qr:], wc)
+            page, off = self._place(slot, pos)
+            self.pages[layer][page, off] = c
+            return norm(lat[:, :qr], wq), c
+        cq = torch.empty(N, qr, dtype=self.dtype, device=lat.device)
+        c = torch.empty(N, R, dtype=self.dtype, device=lat.device) if keep else None
+        a = self._args(layer, slot, pos)
+        _lib.check(_lib.lib().cgk_latent_norm_append(ctypes.byref(a), lat.data_ptr(), int(lat.dtype == torch.float32), lat.stride(0), wq.data_ptr(),
+                                                     wc.data_ptr(), qr, float(eps), cq.data_ptr(), _lib.ptr(c), N, _lib.stream_ptr()),
+                   "cgk_latent_norm_append")
+        _lib.count_launch()
+        return cq, c
+
+    def gather(self, layer: int, slot: int, length: int) -> torch.Tensor:
+        """The first ``length`` latents of the sequence in ``slot``, contiguous."""
+        if self.device.type != "cuda":
+            pos = torch.arange(length)
+            page, off = self._place(torch.full_like(pos, slot), pos)
+            return self.pages[layer][page, off]
+        out = torch.empty(length, self.ranks[layer], dtype=self.dtype, device=self.device)
+        a = self._args(layer)
+        _lib.check(_lib.lib().cgk_latent_gather(ctypes.byref(a), slot, length, out.data_ptr(), _lib.stream_ptr()), "cgk_latent_gather")
+        _lib.count_launch()
+        return out
+
+    def attention(self, layer: int, q, slot, pos, scale: float, max_len: int, force_simt: bool = False) -> torch.Tensor:
+        """q [N, H, rank], queries mapped into the latent space; token t stands at pos[t] of the sequence in slot[t]
+        and sees its latents 0 .. pos[t] (all appended).  Returns softmax(scale q c^T) c.  ``max_len`` bounds the
+        sequence lengths (it sizes the key ranges, not the result)."""
+        N, H, R = q.shape
+        if not q.is_cuda:
+            out = torch.empty(N, H, R, dtype=q.dtype)
+            for t in range(N):
+                c = self.gather(layer, int(slot[t]), int(pos[t]) + 1).float()
+                out[t] = (torch.softmax(q[t].float() @ c.T * scale, -1) @ c).to(q.dtype)
+            return out
+        L = _lib.lib()
+        out = torch.empty_like(q)
+        splits = 1
+        if q.dtype == torch.bfloat16 and not force_simt and L.cgk_latent_attention_tc_ok(R, self.page_size, H):
+            # CTAs per key range: one per token and group of up to 32 heads; ranges of at least two 128-key blocks
+            groups = (H + 31) // 32
+            splits = max(1, min(32, 296 // max(1, N * groups), (max_len + 255) // 256))
+        need = L.cgk_latent_attention_scratch_floats(N, H, R, splits)
+        scratch = torch.empty(need, dtype=torch.float32, device=q.device) if need else None
+        a = self._args(layer, slot, pos, H, scale)
+        _lib.check(L.cgk_latent_attention(ctypes.byref(a), q.data_ptr(), out.data_ptr(), N, splits, _lib.ptr(scratch), int(force_simt),
+                                          _lib.stream_ptr()), "cgk_latent_attention")
+        _lib.count_launch(2 if splits > 1 else 1)
         return out

@@ -44,6 +44,10 @@ struct GemmDev {
   // out_fp32 && accumulate and no other epilogue term).  For weight gradients: a small
   // output with a very long reduction dimension gives too few tiles for the SMs otherwise.
   int split_k, kb_per_split;
+  // Grouped product (mixture of experts): row tile tm multiplies matrix m_group[tm] of the B batch, and only
+  // the first *m_count row tiles exist (both written by an earlier kernel on the same stream).
+  const int* m_group;
+  const int* m_count;
   // ---- hooks used by the fused kernels (all off when zero / null) ----
   // A-operand readiness: before loading rows [m0, m0+128) of A the producer waits
   // until a_ready[m0 / a_ready_rows] >= a_ready_target (flags set by the copy CTAs
@@ -150,8 +154,9 @@ struct GemmSmem {
   static_assert(TOTAL <= 227 * 1024, "GEMM: shared memory budget of one CTA exceeded");
 };
 
-__device__ __forceinline__ void tile_coords(const GemmDev& g, int t, int& b, int& tm, int& tn) {
-  const int per_batch = g.tiles_m * g.tiles_n;
+// tiles_m: g.tiles_m, or the number of row tiles in use (grouped product)
+__device__ __forceinline__ void tile_coords(const GemmDev& g, int tiles_m, int t, int& b, int& tm, int& tn) {
+  const int per_batch = tiles_m * g.tiles_n;
   b = t / per_batch;
   int r = t - b * per_batch;
   if (g.rs_ranks > 0 || g.a_ready) {
@@ -163,7 +168,7 @@ __device__ __forceinline__ void tile_coords(const GemmDev& g, int t, int& b, int
     const int group_sz = GROUP_M * g.tiles_n;
     const int gidx = r / group_sz;
     const int first_m = gidx * GROUP_M;
-    const int rows_in_group = min(GROUP_M, g.tiles_m - first_m);
+    const int rows_in_group = min(GROUP_M, tiles_m - first_m);
     const int rr = r - gidx * group_sz;
     tm = first_m + rr % rows_in_group;
     tn = rr / rows_in_group;
@@ -174,7 +179,7 @@ __device__ __forceinline__ void tile_coords(const GemmDev& g, int t, int& b, int
 
 // cta / nctas: index and count of the CTAs that run this body (the fused kernels
 // give some CTAs of the grid other roles).  GEMM_THREADS threads.
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool GROUPED = false>
 __device__ __forceinline__ void gemm_tc_body(const CUtensorMap& tmA, const CUtensorMap& tmB,
                                              const CUtensorMap* tmC, const CUtensorMap* tmAux,
                                              const CUtensorMap* tmIn,
@@ -223,7 +228,8 @@ __device__ __forceinline__ void gemm_tc_body(const CUtensorMap& tmA, const CUten
   tc_fence_after();
   const uint32_t tmem_base = *tmem_holder;
 
-  const int out_tiles = g.batch * g.tiles_m * g.tiles_n;
+  const int tiles_m = GROUPED ? min(g.tiles_m, *g.m_count) : g.tiles_m;
+  const int out_tiles = g.batch * tiles_m * g.tiles_n;
   const int total_tiles = out_tiles * g.split_k;       // work units: unit u = (split u / out_tiles, tile u % out_tiles)
   const int kblocks_all = (g.K + BK - 1) / BK;
   auto k_range = [&](int u, int& kb0, int& kb1) {
@@ -245,9 +251,10 @@ __device__ __forceinline__ void gemm_tc_body(const CUtensorMap& tmA, const CUten
       int last_ready_chunk = -1;
       for (int t = cta; t < total_tiles && ok; t += nctas) {
         int b, tm, tn, kb0, kb1;
-        tile_coords(g, t % out_tiles, b, tm, tn);
+        tile_coords(g, tiles_m, t % out_tiles, b, tm, tn);
         k_range(t, kb0, kb1);
         const int m0 = tm * BM, n0 = tn * BN;
+        const int bb = GROUPED ? g.m_group[tm] : b;
         if (g.a_ready) {
           // rows of this tile may span two chunks when a_ready_rows < 128: wait for the last one
           const int last_row = min(m0 + BM, g.M) - 1;
@@ -275,11 +282,11 @@ __device__ __forceinline__ void gemm_tc_body(const CUtensorMap& tmA, const CUten
               tma_load_3d(sA + blk * 8192, &tmA, full_bar(s), m0 + blk * 64, kb * BK, b);
           }
           if (!g.b_mn) {
-            tma_load_3d(sB, &tmB, full_bar(s), kb * BK, n0, b);
+            tma_load_3d(sB, &tmB, full_bar(s), kb * BK, n0, bb);
           } else {
 #pragma unroll
             for (int blk = 0; blk < BN / 64; ++blk)
-              tma_load_3d(sB + blk * 8192, &tmB, full_bar(s), n0 + blk * 64, kb * BK, b);
+              tma_load_3d(sB + blk * 8192, &tmB, full_bar(s), n0 + blk * 64, kb * BK, bb);
           }
         }
       }

@@ -27,6 +27,16 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
   gemm_tc_body<BN, STAGES>(tmA, tmB, &tmC, &tmAux, &tmIn, g, (int)blockIdx.x, (int)gridDim.x, smem_raw);
 }
 
+// Grouped product: the rows of A lie in expert order, every expert's segment starts on a row tile, and the
+// number of row tiles is known on the device only.
+template <int BN, int STAGES>
+__global__ void __launch_bounds__(GEMM_THREADS, 1)
+gemm_bf16_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
+                         const __grid_constant__ CUtensorMap tmC, const GemmDev g) {
+  extern __shared__ uint8_t smem_raw[];
+  gemm_tc_body<BN, STAGES, true>(tmA, tmB, &tmC, &tmC, &tmC, g, (int)blockIdx.x, (int)gridDim.x, smem_raw);
+}
+
 // CUDA-core fallback for operands that TMA cannot address (leading dimension not a
 // multiple of 8 elements, unaligned base) and for tiny problems in tests.
 __global__ void gemm_bf16_simt_kernel(const __nv_bfloat16* __restrict__ A,
@@ -216,7 +226,56 @@ static int launch_tc(const cgk_gemm_args& a, const GemmDev& g0, int sms, cudaStr
   return 0;
 }
 
+template <int BN, int STAGES>
+static int launch_grouped(const cgk_gemm_args& a, const GemmDev& g0, int sms, cudaStream_t stream) {
+  using L = GemmSmem<BN, STAGES>;
+  GemmDev g = g0;
+  g.tiles_m = (a.M + BM - 1) / BM;
+  g.tiles_n = (a.N + BN - 1) / BN;
+  CUtensorMap tmA, tmB, tmC, tmAux, tmIn;
+  int rc = make_gemm_tmaps(a, BN, &tmA, &tmB);
+  if (rc) return rc;
+  cgk_gemm_args one = a;
+  one.batch = 1;
+  int out_ok = 0, in_kind = 0;
+  if ((rc = make_gemm_out_tmaps(one, &tmC, &tmAux, &tmIn, &out_ok, &in_kind))) return rc;
+  g.tma_store = out_ok ? 1 : 0;
+  CGK_CUDA_CHECK(cudaFuncSetAttribute(gemm_bf16_grouped_kernel<BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL));
+  const int total = g.tiles_m * g.tiles_n;
+  gemm_bf16_grouped_kernel<BN, STAGES><<<total < sms ? total : sms, GEMM_THREADS, L::TOTAL, stream>>>(tmA, tmB, tmC, g);
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
+
 }  // namespace cgk
+
+CGK_API int cgk_gemm_grouped_bf16(const cgk_gemm_args* pa, const int* tile_group, const int* tiles, void* stream_) {
+  using namespace cgk;
+  CGK_REQUIRE(pa && tile_group && tiles, "cgk_gemm_grouped_bf16: null args");
+  cgk_gemm_args a = *pa;
+  CGK_REQUIRE(a.A && a.B && a.out && a.M >= 0 && a.N >= 0 && a.K > 0 && a.batch >= 1, "cgk_gemm_grouped_bf16: bad arguments");
+  CGK_REQUIRE(!a.a_mn && !a.b_mn && !a.accumulate && !a.bias && !a.act && !a.residual && !a.aux_out && !a.aux_in && !a.rope_cos && a.alpha == 1.0f,
+              "cgk_gemm_grouped_bf16: plain K-major products only");
+  if (a.M == 0 || a.N == 0) return 0;
+  a.strideA = (int64_t)a.M * a.lda;                    // A is one matrix: only its first batch entry is addressed
+  CGK_REQUIRE(gemm_tma_ok(a) && a.M % BM == 0, "cgk_gemm_grouped_bf16: operands must satisfy the TMA alignment rules, rows whole tiles");
+  int dev = 0;
+  CGK_CUDA_CHECK(cudaGetDevice(&dev));
+  GemmDev g;
+  int rc = fill_gemm_dev(a, &g);
+  if (rc) return rc;
+  g.batch = 1;
+  g.m_group = tile_group;
+  g.m_count = tiles;
+  const int sms = sm_count(dev);
+  cgk_gemm_args shape = a;
+  shape.batch = 1;
+  switch (pick_bn(shape, sms)) {
+    case 256: return launch_grouped<256, 4>(a, g, sms, (cudaStream_t)stream_);
+    case 128: return launch_grouped<128, 6>(a, g, sms, (cudaStream_t)stream_);
+    default: return launch_grouped<64, 8>(a, g, sms, (cudaStream_t)stream_);
+  }
+}
 
 CGK_API int cgk_gemm_bf16(const cgk_gemm_args* pa, void* stream_) {
   using namespace cgk;

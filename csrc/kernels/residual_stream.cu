@@ -1,0 +1,194 @@
+// Decoders that keep the residual stream in fp32 and normalise the OUTPUT of a sublayer:
+//   * token embedding times a constant plus a sinusoidal position vector -> fp32 stream + operand copy,
+//   * stream update x += rms(y) * w, where y is a projection's result, or a weighted sum of expert
+//     rows (some of which may stand for the stream itself) plus such a result; the new stream also leaves
+//     as the bf16 (or fp32) operand of the next sublayer,
+//   * RMS norm of selected stream rows (before the vocabulary projection).
+// One CTA per row: a row is read once, kept in shared memory between the statistics and the update.
+#include "../../include/cogito_kernels.h"
+#include "host_common.h"
+#include "sm100.cuh"
+#include "typed_io.cuh"
+
+namespace cgk {
+namespace {
+
+template <typename TE, typename TH>
+__global__ void embed_sinusoid_kernel(const long long* __restrict__ ids, const int* __restrict__ pos, const TE* __restrict__ table,
+                                      float scale, const double* __restrict__ freq, float* __restrict__ x,
+                                      TH* __restrict__ h, int D, int vocab) {
+  const long long row = blockIdx.x;
+  const long long id = CGK_IDX(ids[row], vocab);
+  const double p = (double)pos[row];
+  const int pairs = (D + 1) / 2;
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    float e0 = 0.0f, e1 = 0.0f;
+    if (freq) {
+      // The angle is formed and reduced in double: thousands of radians in fp32 would carry an error of
+      // a few 1e-4, which the fp32 mode of the model would show.
+      const double two_pi = 6.283185307179586;
+      double a = p * freq[i];
+      a -= two_pi * rint(a / two_pi);
+      sincosf((float)a, &e0, &e1);
+    }
+    const int c = 2 * i;
+    const float v0 = ld1(table + id * D + c) * scale + e0;
+    x[row * D + c] = v0;
+    st1(h + row * D + c, v0);
+    if (c + 1 < D) {
+      const float v1 = ld1(table + id * D + c + 1) * scale + e1;
+      x[row * D + c + 1] = v1;
+      st1(h + row * D + c + 1, v1);
+    }
+  }
+}
+
+struct UpdateDev {
+  const void* y; long long ldy;
+  const void* pairs; long long ldp;
+  const int* row_of; const float* weight; int top; int pair_rows;
+  const float* w; float* x; void* h;
+  int D; float eps;
+};
+
+template <typename TY, typename TP, typename TH, int V>
+__global__ void stream_update_kernel(const UpdateDev a) {
+  extern __shared__ float row_buf[];
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  const TY* y = reinterpret_cast<const TY*>(a.y);
+  const TP* pairs = reinterpret_cast<const TP*>(a.pairs);
+  float* x = a.x + t * a.D;
+  float ss = 0.0f;
+  for (int c = threadIdx.x * V; c < a.D; c += blockDim.x * V) {
+    float v[V];
+    if (y) {
+      ldv<V>(y + t * a.ldy + c, v);
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = 0.0f;
+    }
+    for (int k = 0; k < a.top; ++k) {
+      const int r = a.row_of[t * a.top + k];
+      const float wk = a.weight[t * a.top + k];
+      float e[V];
+      if (r >= 0) ldv<V>(pairs + CGK_IDX(r, a.pair_rows) * a.ldp + c, e);
+      else ldv<V>(x + c, e);                          // an expert whose output is its input
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = fmaf(wk, e[j], v[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) { ss = fmaf(v[j], v[j], ss); row_buf[c + j] = v[j]; }
+  }
+  ss = block_sum(ss, red);
+  const float rstd = 1.0f / sqrtf(ss / a.D + a.eps);
+  TH* h = reinterpret_cast<TH*>(a.h) + t * a.D;
+  for (int c = threadIdx.x * V; c < a.D; c += blockDim.x * V) {
+    float xv[V], wv[V];
+    ldv<V>(x + c, xv);
+    ldv<V>(a.w + c, wv);
+#pragma unroll
+    for (int j = 0; j < V; ++j) xv[j] += row_buf[c + j] * rstd * wv[j];
+    stv<V>(x + c, xv);
+    stv<V>(h + c, xv);
+  }
+}
+
+template <typename TO>
+__global__ void rms_rows_kernel(const float* __restrict__ x, const long long* __restrict__ rows, int n_rows, const float* __restrict__ w,
+                                TO* __restrict__ out, int D, float eps) {
+  __shared__ float red[33];
+  const long long i = blockIdx.x;
+  const float* xr = x + CGK_IDX(rows ? rows[i] : i, n_rows) * D;
+  float ss = 0.0f;
+  for (int c = threadIdx.x; c < D; c += blockDim.x) ss = fmaf(xr[c], xr[c], ss);
+  ss = block_sum(ss, red);
+  const float rstd = 1.0f / sqrtf(ss / D + eps);
+  for (int c = threadIdx.x; c < D; c += blockDim.x) st1(out + i * D + c, xr[c] * rstd * w[c]);
+}
+
+// threads for a row of n work items
+int row_threads(int n) { return n <= 64 ? 64 : (n >= 512 ? 512 : (n + 31) / 32 * 32); }
+
+template <typename TY, typename TP, typename TH>
+int launch_update(const UpdateDev& d, int rows, bool vec, cudaStream_t st) {
+  const int smem = d.D * 4;
+  const int nt = row_threads(vec ? d.D / 4 : d.D);
+  if (vec) {
+    if (smem > 48 * 1024)
+      CGK_CUDA_CHECK(cudaFuncSetAttribute(stream_update_kernel<TY, TP, TH, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    stream_update_kernel<TY, TP, TH, 4><<<rows, nt, smem, st>>>(d);
+  } else {
+    if (smem > 48 * 1024)
+      CGK_CUDA_CHECK(cudaFuncSetAttribute(stream_update_kernel<TY, TP, TH, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    stream_update_kernel<TY, TP, TH, 1><<<rows, nt, smem, st>>>(d);
+  }
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
+
+}  // namespace
+}  // namespace cgk
+
+using namespace cgk;
+
+CGK_API int cgk_embed_sinusoid(const void* ids, const void* pos, const void* table, int table_fp32, float scale, const void* freq,
+                               void* x, void* h, int h_fp32, int rows, int D, int vocab, void* stream) {
+  CGK_REQUIRE(ids && pos && table && x && h && rows >= 0 && D > 0 && vocab > 0, "cgk_embed_sinusoid: bad arguments");
+  if (rows == 0) return 0;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int nt = (D + 1) / 2 < 256 ? 128 : 256;
+  const long long* i = (const long long*)ids;
+  const int* p = (const int*)pos;
+  const double* f = (const double*)freq;
+  if (table_fp32 && h_fp32)
+    embed_sinusoid_kernel<float, float><<<rows, nt, 0, st>>>(i, p, (const float*)table, scale, f, (float*)x, (float*)h, D, vocab);
+  else if (!table_fp32 && !h_fp32)
+    embed_sinusoid_kernel<__nv_bfloat16, __nv_bfloat16><<<rows, nt, 0, st>>>(i, p, (const __nv_bfloat16*)table, scale, f, (float*)x,
+                                                                             (__nv_bfloat16*)h, D, vocab);
+  else
+    CGK_REQUIRE(false, "cgk_embed_sinusoid: table and operand copy must have one type");
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
+
+CGK_API int cgk_stream_update(const cgk_stream_update_args* pa, void* stream) {
+  CGK_REQUIRE(pa, "cgk_stream_update: null args");
+  const cgk_stream_update_args& a = *pa;
+  CGK_REQUIRE(a.x && a.h && a.w && a.rows >= 0 && a.D > 0 && (a.y || a.pairs), "cgk_stream_update: bad arguments");
+  CGK_REQUIRE(a.D * 4 <= 200 * 1024, "cgk_stream_update: rows of %d elements are too long", a.D);
+  CGK_REQUIRE(!a.pairs || (a.row_of && a.weight && a.top > 0), "cgk_stream_update: expert rows need their index and weight tables");
+  if (a.rows == 0) return 0;
+  UpdateDev d{a.y, a.ldy, a.pairs, a.ldp, a.row_of, a.weight, a.pairs ? a.top : 0, a.pair_rows, a.w, a.x, a.h, a.D, a.eps};
+  auto ok = [](const void* p, long long ld, int es) { return !p || ((((uintptr_t)p) % (4 * es)) == 0 && ld % 4 == 0); };
+  const bool vec = a.D % 4 == 0 && ok(a.y, a.ldy, a.y_fp32 ? 4 : 2) && ok(a.pairs, a.ldp, a.pairs_fp32 ? 4 : 2) &&
+                   ok(a.x, a.D, 4) && ok(a.w, a.D, 4) && ok(a.h, a.D, a.h_fp32 ? 4 : 2);
+  cudaStream_t st = (cudaStream_t)stream;
+  typedef __nv_bfloat16 bf;
+  if (a.h_fp32) {
+    CGK_REQUIRE((!a.y || a.y_fp32) && (!a.pairs || a.pairs_fp32), "cgk_stream_update: the fp32 form takes fp32 inputs");
+    return launch_update<float, float, float>(d, a.rows, vec, st);
+  }
+  const bool yf = a.y && a.y_fp32, pf = a.pairs && a.pairs_fp32;
+  if (yf && pf) return launch_update<float, float, bf>(d, a.rows, vec, st);
+  if (yf) return launch_update<float, bf, bf>(d, a.rows, vec, st);
+  if (pf) return launch_update<bf, float, bf>(d, a.rows, vec, st);
+  return launch_update<bf, bf, bf>(d, a.rows, vec, st);
+}
+
+CGK_API int cgk_rms_rows(const void* x, const void* rows, int n_out, int n_rows, const void* w, void* out, int out_fp32, int D, float eps,
+                         void* stream) {
+  CGK_REQUIRE(x && w && out && n_out >= 0 && D > 0, "cgk_rms_rows: bad arguments");
+  if (n_out == 0) return 0;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int nt = row_threads(D);
+  if (out_fp32)
+    rms_rows_kernel<float><<<n_out, nt, 0, st>>>((const float*)x, (const long long*)rows, n_rows, (const float*)w, (float*)out, D, eps);
+  else
+    rms_rows_kernel<__nv_bfloat16><<<n_out, nt, 0, st>>>((const float*)x, (const long long*)rows, n_rows, (const float*)w,
+                                                        (__nv_bfloat16*)out, D, eps);
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
+
+CGK_BOUNDS_READER(residual_stream)

@@ -269,6 +269,71 @@ int cgk_softmax_dropout_residual(int dtype, const void* x, const void* mul, cons
 int cgk_softmax_dropout_residual_backward(int dtype, const void* x, const void* mul, const void* dy, void* dx,
                                           int R, int V, float p, unsigned long long seed, void* stream);
 
+/* ---- Decoders with an fp32 residual stream and norms on sublayer outputs (csrc/kernels/residual_stream.cu) ---- */
+/* x[r] = table[ids[r]] * scale + position vector: entry 2i is sin(pos * freq[i]), entry 2i + 1 the cosine
+ * (freq: fp64 [ceil(D / 2)], null = no position vector).  x fp32; h is the same row in the table's type. */
+int cgk_embed_sinusoid(const void* ids, const void* pos, const void* table, int table_fp32, float scale, const void* freq,
+                       void* x, void* h, int h_fp32, int rows, int D, int vocab, void* stream);
+/* v = y[t] + sum_k weight[t, k] * (row_of[t, k] >= 0 ? pairs[row_of[t, k]] : x[t]);
+ * x[t] += v / sqrt(mean(v^2) + eps) * w;  h[t] = x[t].   y or pairs may be null. */
+typedef struct {
+  const void* y; int64_t ldy;
+  const void* pairs; int64_t ldp;
+  const int32_t* row_of; const float* weight;
+  const float* w; float* x; void* h;
+  int32_t rows, D, top, pair_rows;
+  int32_t y_fp32, pairs_fp32, h_fp32;
+  float eps;
+} cgk_stream_update_args;
+int cgk_stream_update(const cgk_stream_update_args* a, void* stream);
+/* out[i] = rms_norm(x[rows[i]]) * w  (rows int64, null = identity; n_rows rows exist). */
+int cgk_rms_rows(const void* x, const void* rows, int n_out, int n_rows, const void* w, void* out, int out_fp32, int D, float eps,
+                 void* stream);
+/* True fp32 product on the CUDA cores: C = A . B^T per batch (b_mn: B stored [K, N]). */
+int cgk_gemm_f32(const void* A, const void* B, void* C, int M, int N, int K, int batch, long long lda, long long ldb, long long ldc,
+                 long long sA, long long sB, long long sC, int b_mn, void* stream);
+
+/* ---- Latent attention (csrc/kernels/latent_kv.cu, latent_attn_tc.cu) ---- */
+/* One layer's paged cache of latents, pages[n_pages][page_size][R] in bf16 (fp32 with `fp32`), and the query
+ * tokens of a call: token t belongs to the sequence in slot[t] and stands at pos[t]. */
+typedef struct {
+  void* pages;
+  const int32_t* page_table;         /* [slots][max_pages] */
+  const int32_t* slot; const int32_t* pos;
+  int32_t R, page_size, max_pages, slots, n_pages, heads, fp32;
+  float scale;
+} cgk_latent_args;
+/* in: [rows][q_rank | R] (ld elements apart).  cq = rms(in[:q_rank]) * wq; c = rms(in[q_rank:]) * wc goes to the
+ * token's cache place and, if c_out is given, to c_out[row]. */
+int cgk_latent_norm_append(const cgk_latent_args* a, const void* in, int in_fp32, long long ld, const void* wq, const void* wc,
+                           int q_rank, float eps, void* cq, void* c_out, int rows, void* stream);
+/* out[p] = latent of position p of `slot`, p < len. */
+int cgk_latent_gather(const cgk_latent_args* a, int slot, int len, void* out, void* stream);
+/* out[t, h] = sum_p softmax_p(scale * q[t, h] . c_p) c_p over the positions p <= pos[t] of the token's sequence;
+ * q, out [rows][heads][R].  splits > 1: key ranges handled by separate CTAs (tensor-core form only). */
+int cgk_latent_attention(const cgk_latent_args* a, const void* q, void* out, int rows, int splits, void* scratch, int force_simt,
+                         void* stream);
+int cgk_latent_attention_tc_ok(int R, int page_size, int heads);
+long long cgk_latent_attention_scratch_floats(int rows, int heads, int R, int splits);
+
+/* ---- Mixture of experts (csrc/kernels/moe.cu) ---- */
+/* scores s = softmax(logits[t]); choice = s + correction; only outputs of the `keep` best of `groups` equal groups
+ * (by largest choice score) can be chosen; idx = the `top` best choices, weight = their s over the sum.  row_of =
+ * t * top + k, or -1 for outputs >= experts (which stand for the input itself).  counts (may be null): += 1 per expert. */
+int cgk_moe_route(const void* logits, const void* correction, int rows, int experts, int outputs, int top, int groups, int keep,
+                  void* idx, void* weight, void* row_of, void* counts, void* stream);
+/* counts -> cursor (first row of an expert's segment, segments start on multiples of 128), tile_expert, *tiles; clears counts. */
+int cgk_moe_plan(void* counts, int experts, void* cursor, void* tile_expert, void* tiles, int max_tiles, void* stream);
+int cgk_moe_gather(const void* h, const void* idx, int pairs, int top, int experts, void* cursor, void* row_of, void* out, int D,
+                   int max_rows, void* stream);
+/* g: A [rows][K] in expert order, B [experts][N][K], out bf16 or fp32 [rows][N]; g->M = allocated rows (a multiple of 128). */
+int cgk_gemm_grouped_bf16(const cgk_gemm_args* g, const int* tile_group, const int* tiles, void* stream);
+int cgk_swiglu_tiles(const void* gate_up, void* act, const void* tiles, int F, int max_tiles, void* stream);
+/* Expert products pair by pair: act [pairs][F] in the weights' type, y fp32 [pairs][D]; w_gate_up [experts][2F][D], w_down
+ * [experts][D][F].  Pairs whose output is not an expert are left alone. */
+int cgk_expert_rows(int fp32, const void* h, const void* idx, int pairs, int top, int experts, const void* w_gate_up, const void* w_down,
+                    void* act, void* y, int D, int F, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
