@@ -104,7 +104,7 @@ class StackEngine:
         if self.use_graph and keep is None and all(len(t) == 1 for _, t, _ in entries):
             logits = self._decode_graph(entries)
             rows = [i for i, (_, _, w) in enumerate(entries) for _ in w]
-            out = logits[torch.tensor(rows, device=self.device)] if rows != list(range(len(entries))) else logits.clone()
+            out = logits[torch.tensor(rows, dtype=torch.int64, device=self.device)] if rows != list(range(len(entries))) else logits.clone()
         else:
             # prompt portions first; the caller's order of the wanted logits is kept by the row list
             order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]) < self.PROMPT_MIN)
