@@ -18,6 +18,7 @@ _SUBPACKAGES = ("nn", "ops", "optim", "models", "parallel", "quant", "serve", "j
 _NAMES = {
     # models
     "GPT2": "models.gpt2", "GPT2Config": "models.gpt2", "Llama": "models.llama", "LlamaConfig": "models.llama",
+    "Surelorn": "models.surelorn", "SurelornConfig": "models.surelorn", "load_folder": "models.registry",
     "MLPClassifier": "models.mlp", "XorNet": "models.mlp", "ConvClassifier": "models.cnn",
     # training
     "Trainer": "train", "FusedAdam": "optim.fused", "FusedSGD": "optim.fused", "GradScaler": "optim.fused",
@@ -27,6 +28,7 @@ _NAMES = {
     # quantisation and serving
     "quantize_int4": "quant.int4", "dequantize_int4": "quant.int4", "Int4Linear": "quant.int4",
     "PagedKVCacheInt4": "serve.kv_cache", "LlamaInt4Engine": "serve.engine", "SpeculativeDecoder": "serve.engine",
+    "PagedLatentCache": "serve.kv_cache", "StackEngine": "serve.stack", "Scheduler": "serve.scheduler", "generate": "serve.scheduler",
     # checkpoints, profiling, failure detection, JIT
     "save_model": "io.checkpoint", "load_model": "io.checkpoint", "save_training_state": "io.checkpoint",
     "load_training_state": "io.checkpoint", "Profiler": "utils.profiler", "instrument": "utils.profiler",

@@ -2,7 +2,9 @@
 
     train     run a training job described by a YAML config (see ``DEFAULTS``): GPT-2, Llama, MLP or
               convolutional classifier; data / tensor / pipeline / 3-D parallel under a launcher
-    generate  INT4 speculative decoding with a draft / target pair (tensor parallel under a launcher)
+    generate  with model.path=FOLDER: the model in that folder (its class is named by config.json), continuous batching
+              over prompts of any lengths; otherwise INT4 speculative decoding with a draft / target Llama pair
+              (tensor parallel under a launcher)
     info      versions, device, library status
 
 A config is a nested mapping; ``section.key=value`` arguments override it (``train.steps=20``,
@@ -88,6 +90,7 @@ def _device(cfg):
 def cmd_train(cfg):
     from .data.datasets import BatchIterator, SyntheticTokens, load_mnist
     from .io import checkpoint as ckpt
+    from .models import registry
     from .optim.fused import FusedAdam, FusedSGD, GradScaler, exp_lr, step_lr
     from .train import Trainer
     from .utils import rng
@@ -108,11 +111,9 @@ def cmd_train(cfg):
     step_fn, model, opt = None, None, None
     logger = rank == 0
     if family == "llama" and world > 1:
-        from .models.llama import LlamaConfig
         from .parallel.groups import init_parallel
         from .parallel.llama_parallel import Trainer3D
-        lc = LlamaConfig(vocab_size=m["vocab_size"], n_layer=m["n_layer"], d_model=m["d_model"], n_head=m["n_head"],
-                         n_kv_head=m["n_kv_head"] or m["n_head"], d_ff=m["d_ff"], max_seq_len=m["max_seq_len"])
+        lc = registry.train_config(family, m)
         ctx = init_parallel(p["dp"], p["tp"], p["pp"])
         mb = t["micro_batch"] or 1
         t3 = Trainer3D(lc, ctx, dev, p["microbatches"], mb, t["seq_len"], lr=t["lr"], loss_scale=t["loss_scale"] if scaler_on else None,
@@ -125,32 +126,13 @@ def cmd_train(cfg):
         c = ctx.coords
         logger = c.pp_rank == c.pp - 1 and c.dp_rank == 0 and c.tp_rank == 0
     else:
-        if family == "gpt2":
-            from .models.gpt2 import GPT2, GPT2Config
-            gc = GPT2Config(vocab_size=m["vocab_size"], n_layer=m["n_layer"], d_model=m["d_model"], n_head=m["n_head"], d_ff=m["d_ff"],
-                            max_seq_len=m["max_seq_len"])
-            if p["tp"] > 1:
-                from .parallel.tensor_parallel import build_tp_gpt2
-                model, sync = build_tp_gpt2(gc, rank, world, dev, micro_tokens=(t["micro_batch"] or t["batch"]) * t["seq_len"])
-                params, parallel = model._ordered, sync
-            else:
-                model = GPT2(gc, device=dev, dtype=dtype)
-                params, parallel = list(model.parameters()), None
-        elif family == "llama":
-            from .models.llama import Llama, LlamaConfig
-            model = Llama(LlamaConfig(vocab_size=m["vocab_size"], n_layer=m["n_layer"], d_model=m["d_model"], n_head=m["n_head"],
-                                      n_kv_head=m["n_kv_head"] or m["n_head"], d_ff=m["d_ff"], max_seq_len=m["max_seq_len"]), device=dev, dtype=dtype)
-            params, parallel = list(model.parameters()), None
-        elif family == "mlp":
-            from .models.mlp import MLPClassifier
-            model = MLPClassifier(m["in_features"], m["hidden"], m["classes"], device=dev, dtype=dtype)
-            params, parallel = list(model.parameters()), None
-        elif family == "cnn":
-            from .models.cnn import ConvClassifier
-            model = ConvClassifier(m["in_channels"], m["image"], m["channels"], m["classes"], device=dev, dtype=dtype)
-            params, parallel = list(model.parameters()), None
+        if family == "gpt2" and p["tp"] > 1:
+            from .parallel.tensor_parallel import build_tp_gpt2
+            model, sync = build_tp_gpt2(registry.train_config(family, m), rank, world, dev, micro_tokens=(t["micro_batch"] or t["batch"]) * t["seq_len"])
+            params, parallel = model._ordered, sync
         else:
-            raise SystemExit(f"unknown model.family {family}")
+            model = registry.train_model(family, m, dev, dtype)
+            params, parallel = list(model.parameters()), None
         scaler = GradScaler(dev, enabled=scaler_on, init_scale=t["loss_scale"] or 1.0)
         kw = dict(lr=t["lr"], weight_decay=t["weight_decay"], scaler=scaler, max_grad_norm=t["max_grad_norm"])
         if p["dp"] > 1 and p["tp"] == 1:
@@ -315,8 +297,57 @@ def cmd_train(cfg):
     return last
 
 
+def cmd_generate_folder(cfg):
+    """``model.path``: a folder with config.json and model.safetensors.  generate.prompts: a JSON list of token-id lists
+    (default: ``batch`` random prompts of ``prompt_len``); new_tokens, temperature (0: greedy), top_k, top_p; slots (live
+    sequences), step_tokens (tokens per engine step); dtype bfloat16 / float32; draft_path: a second folder whose model
+    drafts for this one (speculative decoding; prompts of equal length); out: file for the sequences."""
+    from .models.registry import load_folder
+    from .serve.scheduler import Scheduler
+    from .serve.stack import StackEngine
+    if int(os.environ.get("WORLD_SIZE", 1)) > 1:
+        raise SystemExit("model.path: folders are served by one process")
+    dev, g = _device(cfg), cfg.get("generate", {})
+    model = load_folder(cfg["model"]["path"], dev, getattr(torch, g.get("dtype", "bfloat16")))
+    new = g.get("new_tokens", 32)
+    if g.get("prompts"):
+        with open(g["prompts"]) as f:
+            prompts = json.load(f)
+    else:
+        prompts = torch.randint(0, model.vocab(), (g.get("batch", 4), g.get("prompt_len", 16)),
+                                generator=torch.Generator().manual_seed(cfg["seed"])).tolist()
+    longest = max(len(p) for p in prompts) + new
+    sampling = dict(temperature=g.get("temperature", 0.0), top_k=g.get("top_k", 0), top_p=g.get("top_p", 1.0), seed=cfg["seed"])
+    if g.get("draft_path"):
+        from .serve.engine import SpeculativeDecoder
+        gamma = g.get("gamma", 4)
+        cap = longest + (gamma + 1) * (new + 1)            # a sequence whose drafts are all accepted runs ahead of the others
+        draft = load_folder(g["draft_path"], dev, model.dtype)
+        dec = SpeculativeDecoder(StackEngine(draft, len(prompts), cap), StackEngine(model, len(prompts), cap), gamma=gamma, **sampling)
+        t0 = time.time()
+        seqs, stats = dec.generate(torch.tensor(prompts, device=dev), new)
+        out = {"generated": stats.generated, "steps": stats.steps, "acceptance_rate": round(stats.acceptance_rate, 4)}
+    else:
+        slots = min(g.get("slots", 32), len(prompts))
+        s = Scheduler(StackEngine(model, slots, longest, pool_tokens=slots * longest), step_tokens=g.get("step_tokens", 2048), **sampling)
+        reqs = [s.add(p, new) for p in prompts]
+        t0 = time.time()
+        s.run()
+        seqs = [r.prompt + r.tokens for r in reqs]
+        out = {"generated": sum(len(r.tokens) for r in reqs), "steps": s.steps}
+    out["tok_per_s"] = round(out["generated"] / (time.time() - t0), 1)
+    if g.get("out"):
+        with open(g["out"], "w") as f:
+            json.dump(seqs, f)
+    print(json.dumps(out))
+    return out
+
+
 def cmd_generate(cfg):
-    from .models.llama import Llama, LlamaConfig
+    if cfg["model"].get("path"):
+        return cmd_generate_folder(cfg)
+    from .models import registry
+    from .models.llama import Llama
     from .serve.engine import LlamaInt4Engine, SpeculativeDecoder
     from .utils import rng
     dev = _device(cfg)
@@ -330,10 +361,8 @@ def cmd_generate(cfg):
     m = cfg["model"]
     g = cfg.get("generate", {})
     dtype = torch.bfloat16 if dev.type == "cuda" else None
-    tc = LlamaConfig(vocab_size=m["vocab_size"], n_layer=m["n_layer"], d_model=m["d_model"], n_head=m["n_head"],
-                     n_kv_head=m["n_kv_head"] or m["n_head"], d_ff=m["d_ff"], max_seq_len=m["max_seq_len"])
-    dc = LlamaConfig(vocab_size=m["vocab_size"], n_layer=g.get("draft_layers", 2), d_model=m["d_model"], n_head=m["n_head"],
-                     n_kv_head=m["n_kv_head"] or m["n_head"], d_ff=m["d_ff"], max_seq_len=m["max_seq_len"])
+    tc = registry.train_config("llama", m)
+    dc = registry.train_config("llama", {**m, "n_layer": g.get("draft_layers", 2)})
     B, L, new = g.get("batch", 4), g.get("prompt_len", 16), g.get("new_tokens", 32)
     if g.get("prompts"):                                          # a JSON list of B token-id lists of equal length
         with open(g["prompts"]) as f:

@@ -15,7 +15,7 @@ import torch
 from .sampling import sample
 
 
-@dataclass
+@dataclass(eq=False)
 class Request:
     prompt: list[int]
     max_new_tokens: int
