@@ -52,8 +52,10 @@ class SurelornConfig:
             mixer = LatentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["q_rank"]), int(m["kv_rank"]), float(m["scale"]))
             layers.append(LayerSpec(mixer, cls._mlp(i, mlp), e.get("weights_of")))
         cfg = cls(int(d["vocab"]), int(d["width"]), tuple(layers), float(d["embedding"]["scale"]), float(d["norm"]["eps"]))
-        for i in range(len(layers)):
-            cfg.home(i)
+        for i, l in enumerate(layers):
+            h = layers[cfg.home(i)]
+            if (l.mixer, l.mlp) != (h.mixer, h.mlp):
+                raise ValueError(f"layer {i} uses the weights of layer {cfg.home(i)}, whose sizes differ")
         return cfg
 
     @staticmethod

@@ -127,6 +127,8 @@ def test_configuration_round_trip_and_rejections(tmp_path):
         SurelornConfig.from_dict({**d, "layers": [S.layer(d["layers"][0]["mixer"], S.moe(8, 6, 3, 2, (4, 1)))]})
     with pytest.raises(ValueError, match="weights_of"):
         SurelornConfig.from_dict({**d, "layers": [S.layer(d["layers"][0]["mixer"], None, 0)]})
+    with pytest.raises(ValueError, match="sizes differ"):
+        SurelornConfig.from_dict({**d, "layers": [d["layers"][0], S.layer(d["layers"][0]["mixer"], None, 0)]})
     t = random_tensors(cfg)
     save_folder(str(tmp_path / "m"), cfg, t)
     back = load_safetensors(str(tmp_path / "m" / "model.safetensors"))

@@ -287,7 +287,7 @@ def test_batches_of_unequal_sequences_and_pages_used_again(dtype):
 
 def test_long_decoding_and_far_keys_in_fp32():
     """700 tokens, most of them decoded one by one: in fp32 a single lost or extra key among hundreds is visible."""
-    d = S.config(48, 60, [S.layer(S.mixer(2, 16, 16, 24, 40, 0.6), S.dense(32)), S.layer(S.mixer(2, 16, 16, 24, 40, 0.6), None, 0)])
+    d = S.config(48, 60, [S.layer(S.mixer(2, 16, 16, 24, 40, 0.6), S.dense(32)), S.layer(S.mixer(2, 16, 16, 24, 40, 0.6), S.dense(32), 0)])
     cfg = S.SurelornConfig.from_dict(d)
     t = S.random_tensors(cfg, 2)
     toks = S.tokens(700, 60, 3)
