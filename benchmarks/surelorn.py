@@ -136,7 +136,7 @@ def kernel_part(width, iters=20):
     from cogito_b200.ops import moe as X
     from cogito_b200.ops import stream as R
     from cogito_b200.ops.attention import flash_forward
-    from cogito_b200.ops.gemm import gemm
+    from cogito_b200.ops.linear import gated_linear, linear
     from cogito_b200.ops.norm import norm_forward_raw
     from cogito_b200.quant.int4 import Int4Linear
     from cogito_b200.serve.kv_cache import PagedKVCacheInt4, PagedLatentCache
@@ -153,11 +153,13 @@ def kernel_part(width, iters=20):
 
     def product(name, like, M_, N_, K_, out=BF):
         a, b = mk(M_, K_), mk(N_, K_)
-        put(name, like, lambda: gemm(a, b, out_dtype=out), 2 * (M_ * K_ + N_ * K_) + (4 if out == torch.float32 else 2) * M_ * N_, 2.0 * M_ * N_ * K_,
+        put(name, like, lambda: linear(a, b, out_dtype=out), 2 * (M_ * K_ + N_ * K_) + (4 if out == torch.float32 else 2) * M_ * N_, 2.0 * M_ * N_ * K_,
             shape=[M_, N_, K_])
 
     with torch.no_grad():
         T = 4096
+        one = torch.zeros(1, device="cuda")
+        put("smallest launch (what the method itself costs)", "-", lambda: one.add_(1))
         # ---- prompt: row kernels
         x, y, w = mk(T, width, dt=torch.float32), mk(T, width), torch.ones(width, device="cuda")
         put("stream_update", "norm", lambda: R.stream_update(x, y, w, 1e-6, BF), T * width * (2 + 4 + 4 + 2))
@@ -171,11 +173,11 @@ def kernel_part(width, iters=20):
         cache = PagedLatentCache([R_], 2, T, 64, "cuda", BF)
         slot = torch.zeros(T, device="cuda", dtype=torch.int32)
         wq, wc = torch.ones(q, device="cuda"), torch.ones(R_, device="cuda")
-        lat = mk(T, q + R_)
-        put("latent_norm_append", "norm", lambda: cache.norm_append(0, lat, wq, wc, 1e-6, slot, pos, True), T * ((q + R_) * 2 + q * 2 + R_ * 4))
+        lat = mk(T, q + R_, dt=torch.float32)
+        put("latent_norm_append", "norm", lambda: cache.norm_append(0, lat, wq, wc, 1e-6, slot, pos, True), T * ((q + R_) * 4 + q * 2 + R_ * 4))
         put("latent_gather", "norm", lambda: cache.gather(0, 0, T), T * R_ * 4)
         # ---- prompt: products and attention
-        product("gemm dq|dkv", "gemm", T, q + R_, width)
+        product("gemm dq|dkv (fp32 out)", "gemm", T, q + R_, width, torch.float32)
         product("gemm uq", "gemm", T, H * D, q)
         product("gemm uk|uv", "gemm", T, 2 * H * D, R_)
         product("gemm o", "gemm", T, width, H * D)
@@ -191,7 +193,7 @@ def kernel_part(width, iters=20):
         # ---- prompt: mixture
         E, top, F = s["experts"], s["top"], s["expert_ff"]
         h, wr = mk(T, width), mk(E, width)
-        put("gemm router", "gemm", lambda: gemm(h, wr, out_dtype=torch.float32), 2 * (T * width + E * width) + 4 * T * E, 2.0 * T * E * width, shape=[T, E, width])
+        put("gemm router", "gemm", lambda: linear(h, wr, out_dtype=torch.float32), 2 * (T * width + E * width) + 4 * T * E, 2.0 * T * E * width, shape=[T, E, width])
         logits, corr = mk(T, E, dt=torch.float32), torch.zeros(E, device="cuda")
         put("moe_route", "sample", lambda: X.route(logits, corr, E, top, 8, 4), T * E * 4 + T * top * 12)
         wgu, wdn = mk(E, 2 * F, width) * width ** -0.5, mk(E, width, F) * F ** -0.5
@@ -216,12 +218,13 @@ def kernel_part(width, iters=20):
         del rows_y, wgu, wdn
         # ---- decode
         for B in (1, 16, 64):
-            product(f"decode gemm dq|dkv ({B})", "decode gemm", B, q + R_, width)
-            product(f"decode gemm gate|up ({B})", "decode gemm", B, 2 * ff, width)
+            product(f"decode gemm dq|dkv ({B})", "decode gemm", B, q + R_, width, torch.float32)
+            ag, wg = mk(B, width), mk(2 * ff, width)
+            put(f"decode gate|up with swiglu ({B})", "decode gemm", lambda: gated_linear(ag, wg), 2 * (B * width + 2 * ff * width + B * ff), 4.0 * B * ff * width)
             product(f"decode gemm down ({B})", "decode gemm", B, width, ff)
             product(f"decode gemm head ({B})", "decode gemm", B, VOCAB, width, torch.float32)
             qh, wk, qa = mk(B, H, D), mk(H, D, R_), mk(B, H, R_)
-            put(f"decode product W_uk^T q ({B})", "decode gemm", lambda: gemm(qh.transpose(0, 1), wk, b_mn=True, out=qa.transpose(0, 1)), 2 * H * D * R_ + 2 * B * H * (D + R_))
+            put(f"decode product W_uk^T q ({B})", "decode gemm", lambda: linear(qh.transpose(0, 1), wk, w_mn=True, out=qa.transpose(0, 1)), 2 * H * D * R_ + 2 * B * H * (D + R_))
             lc = PagedLatentCache([R_], B, CONTEXT, 64, "cuda", BF)
             lc.pages[0].normal_()
             p1 = torch.full((B,), CONTEXT - 1, device="cuda", dtype=torch.int32)

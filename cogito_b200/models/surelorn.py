@@ -20,7 +20,7 @@ from torch import nn
 from ..nn.latent_attention import LatentAttention, LatentSpec, _frozen
 from ..nn.moe import DenseSpec, GatedMLP, MixtureOfExperts, MoESpec
 from ..ops import stream as S
-from ..ops.gemm import gemm
+from ..ops.linear import linear
 
 POSITION_BASE = 10000.0
 
@@ -211,7 +211,7 @@ class Surelorn(nn.Module):
 
     def logits(self, x: torch.Tensor, rows: torch.Tensor | None = None) -> torch.Tensor:
         """fp32 logits of the stream's rows (all, or those named)."""
-        return gemm(S.rms_rows(x, self.norm_f, self.cfg.norm_eps, self.dtype, rows), self.head, out_dtype=torch.float32)
+        return linear(S.rms_rows(x, self.norm_f, self.cfg.norm_eps, self.dtype, rows), self.head, out_dtype=torch.float32)
 
     def num_params(self) -> int:
         return sum(p.numel() for p in self.parameters())

@@ -17,7 +17,7 @@ import torch
 from torch import nn
 
 from ..ops.attention import flash_forward
-from ..ops.gemm import gemm
+from ..ops.linear import linear
 
 
 @dataclass(frozen=True)
@@ -85,7 +85,7 @@ class LatentAttention(nn.Module):
         else:
             length = seg.begin + seg.count
             ctx = cache.gather(layer, seg.slot, length)
-        kv = gemm(ctx, self.w_ukv).view(seg.sequences, length, 2, H, self.dq)
+        kv = linear(ctx, self.w_ukv).view(seg.sequences, length, 2, H, self.dq)
         shape = (seg.sequences, seg.count, H, self.dq)
         flash_forward(q[lo:lo + n].view(shape), kv[:, :, 0], kv[:, :, 1], causal=True, scale=s.scale, out=out[lo:lo + n].view(shape))
 
@@ -96,22 +96,22 @@ class LatentAttention(nn.Module):
         wv = self.w_ukv[H * self.dq:].view(H, self.dv, R)
         qh = q[lo:].view(n, H, self.dq).transpose(0, 1)
         qa = torch.empty(n, H, R, dtype=q.dtype, device=q.device)
-        gemm(qh, wk, b_mn=True, out=qa.transpose(0, 1))
+        linear(qh, wk, w_mn=True, out=qa.transpose(0, 1))
         ol = cache.attention(layer, qa, batch.slot[lo:], batch.pos[lo:], s.scale, batch.max_len)
-        gemm(ol.transpose(0, 1), wv, out=out[lo:].view(n, H, self.dv).transpose(0, 1))
+        linear(ol.transpose(0, 1), wv, out=out[lo:].view(n, H, self.dv).transpose(0, 1))
 
     def forward(self, h: torch.Tensor, batch, cache, layer: int) -> torch.Tensor:
         """h [N, width], the tokens of ``batch``; appends their latents to layer ``layer`` of ``cache``."""
         s = self.spec
-        lat = gemm(h, self.w_down, out_dtype=torch.float32)
+        lat = linear(h, self.w_down, out_dtype=torch.float32)
         segs = batch.prompts if self.prompt_form else ()
         split = batch.single_from if self.prompt_form else 0
         cq, c = cache.norm_append(layer, lat, self.q_norm, self.kv_norm, self.eps, batch.slot, batch.pos,
                                   keep=any(seg.begin == 0 for seg in segs))
-        q = gemm(cq, self.w_uq)
+        q = linear(cq, self.w_uq)
         o = torch.empty(h.shape[0], s.heads * self.dv, dtype=h.dtype, device=h.device)
         for seg in segs:
             self._expanded(q, seg, layer, cache, c, o)
         if split < h.shape[0]:
             self._latent(q, split, batch, layer, cache, o)
-        return gemm(o, self.w_o)
+        return linear(o, self.w_o)

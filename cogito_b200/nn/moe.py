@@ -8,9 +8,8 @@ from dataclasses import dataclass
 import torch
 from torch import nn
 
-from ..ops import misc as M
 from ..ops import moe as X
-from ..ops.gemm import gemm
+from ..ops.linear import gated_linear, linear
 from .latent_attention import _frozen
 
 
@@ -35,7 +34,7 @@ class MoESpec:
 
 
 class GatedMLP(nn.Module):
-    """W_down (silu(W_gate h) * (W_up h)); the gate and up products are one GEMM."""
+    """W_down (silu(W_gate h) * (W_up h)); the gate and up products are one product."""
 
     def __init__(self, tensors, device, dtype):
         super().__init__()
@@ -44,7 +43,7 @@ class GatedMLP(nn.Module):
         self.w_down = _frozen(t["down"].to(dtype).contiguous())
 
     def forward(self, h):
-        return gemm(M.swiglu(gemm(h, self.w_gate_up)), self.w_down)
+        return linear(gated_linear(h, self.w_gate_up), self.w_down)
 
     def branch(self, h):
         """What the stream update adds: (dense result, no expert rows)."""
@@ -67,7 +66,7 @@ class MixtureOfExperts(nn.Module):
     def branch(self, h):
         """(shared expert's result or None, the weighted expert rows as keyword arguments of ``stream_update``)."""
         s = self.spec
-        logits = gemm(h, self.w_router, out_dtype=torch.float32)
+        logits = linear(h, self.w_router, out_dtype=torch.float32)
         grouped = X.grouped_ok(h, self.w_gate_up, self.w_down) and h.shape[0] * s.top > X.FEW_PAIRS
         r = X.route(logits, self.correction, s.experts, s.top, s.groups, s.keep, count=grouped)
         rows = X.expert_outputs(h, r, self.w_gate_up, self.w_down)

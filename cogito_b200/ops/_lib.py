@@ -108,6 +108,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_stream_update": [vp, vp],
         "cgk_rms_rows": [vp, vp, i, i, vp, vp, i, i, f, vp],
         "cgk_gemm_f32": [vp, vp, vp, i, i, i, i, ll, ll, ll, ll, ll, ll, i, vp],
+        "cgk_skinny_gemm": [vp, ll, ll, vp, ll, ll, vp, ll, ll, i, i, i, i, i, i, vp],
         "cgk_latent_norm_append": [vp, vp, i, ll, vp, vp, i, f, vp, vp, i, vp],
         "cgk_latent_gather": [vp, i, i, vp, vp],
         "cgk_latent_attention": [vp, vp, vp, i, i, vp, i, vp],

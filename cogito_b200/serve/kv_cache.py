@@ -285,9 +285,9 @@ class PagedLatentCache(PagedCache):
         out = torch.empty_like(q)
         splits = 1
         if q.dtype == torch.bfloat16 and not force_simt and L.cgk_latent_attention_tc_ok(R, self.page_size, H):
-            # CTAs per key range: one per token and group of up to 32 heads; ranges of at least two 128-key blocks
+            # CTAs per key range: one per token and group of up to 32 heads; ranges of whole 128-key blocks
             groups = (H + 31) // 32
-            splits = max(1, min(32, 296 // max(1, N * groups), (max_len + 255) // 256))
+            splits = max(1, min(32, 148 // max(1, N * groups), (max_len + 127) // 128))
         need = L.cgk_latent_attention_scratch_floats(N, H, R, splits)
         scratch = torch.empty(need, dtype=torch.float32, device=q.device) if need else None
         a = self._args(layer, slot, pos, H, scale)

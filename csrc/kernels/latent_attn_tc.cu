@@ -6,9 +6,11 @@
 //      a ring, so those of the next block arrive while this block's products run,
 //   2. S^T[128 keys, NP] = C . Q^T          (tcgen05.mma by warp 9, keys on the TMEM lanes),
 //   3. warps 0..7: scale, mask, row maxima through a row-major copy in shared memory, p = 2^(s - m); p is
-//      stored as the sum of two bf16 numbers, so the product below sees the weight to 16 bits,
-//   4. O^T[R, NP] += C^T . P^T              (the same slices read MN-major); O stays in TMEM and is rescaled
-//      only when a row maximum grows by more than 2^8.  A slice goes back to the ring when its product is done.
+//      stored as the sum of two bf16 numbers (two column groups of one operand tile), so the product below sees
+//      the weight to 16 bits at the price of a wider instruction,
+//   4. O^T[R, 2 NP] += C^T . P^T            (the same slices read MN-major); O stays in TMEM, is rescaled only
+//      when a row maximum grows by more than 2^8, and its two column groups are added at the end.  A slice goes back
+//      to the ring when its product is done.
 // The kernel is bound by reading the latents (R * 2 bytes per key for all heads of the group).
 #include "../../include/cogito_kernels.h"
 #include "host_common.h"
@@ -113,7 +115,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
   volatile int* go = reinterpret_cast<volatile int*>(sm + o_misc + 8);
   volatile int* grew = reinterpret_cast<volatile int*>(sm + o_misc + 12);
   uint32_t cols = 32;
-  while (cols < (uint32_t)(NP * (ns + 1))) cols <<= 1;
+  while (cols < (uint32_t)(NP * (2 * ns + 1))) cols <<= 1;
 
   if (tid == 0) {
     for (int s = 0; s < slots; ++s) { mbar_init(full_bar(s), 1); mbar_init(empty_bar(s), 1); }
@@ -170,7 +172,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
     }
   } else if (warp == 9) {
     if (lane == 0) {
-      const uint32_t id_s = make_idesc_bf16(128, NP, 0, 0), id_o = make_idesc_bf16(128, NP, 1, 0);
+      const uint32_t id_s = make_idesc_bf16(128, NP, 0, 0), id_o = make_idesc_bf16(128, 2 * NP, 1, 0);
       bool ok = true;
       for (int b = 0; b < nblk && ok; ++b) {
         for (int m = 0; m < ns; ++m) {
@@ -190,12 +192,9 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
         for (int m = 0; m < ns; ++m) {
           const int it = b * ns + m, s = it % slots;
 #pragma unroll
-          for (int part = 0; part < 2; ++part)
-#pragma unroll
-            for (int kk = 0; kk < LT_KB / 16; ++kk)
-              umma_f16(tmem + NP * (1 + m), make_smem_desc_sw128(sb + s * LT_SLICE + kk * 2048, 16384, 1024),
-                       make_smem_desc_sw128(sb + o_t + part * (NP * 256) + (kk >> 2) * (NP * 128) + (kk & 3) * 32, 16, 1024), id_o,
-                       b != 0 || part != 0 || kk != 0);
+          for (int kk = 0; kk < LT_KB / 16; ++kk)
+            umma_f16(tmem + NP * (1 + 2 * m), make_smem_desc_sw128(sb + s * LT_SLICE + kk * 2048, 16384, 1024),
+                     make_smem_desc_sw128(sb + o_t + (kk >> 2) * (NP * 256) + (kk & 3) * 32, 16, 1024), id_o, b != 0 || kk != 0);
           umma_commit(empty_bar(s));
         }
         if (b + 1 == nblk) umma_commit(o_full);
@@ -255,7 +254,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
       }
       lt_meet();
       float corr[CPT];
-      uint8_t* pbase = sm + o_t + (kin >> 6) * (NP * 128) + (kin & 7) * 2;
+      uint8_t* pbase = sm + o_t + (kin >> 6) * (NP * 256) + (kin & 7) * 2;
 #pragma unroll
       for (int j = 0; j < CPT; ++j) {
         const int r = half * CPT + j;
@@ -265,11 +264,11 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
         const __nv_bfloat16 hi = __float2bfloat16(p);
         const uint32_t off = sw128_offset(r, (kin & 63) >> 3);
         *reinterpret_cast<__nv_bfloat16*>(pbase + off) = hi;
-        *reinterpret_cast<__nv_bfloat16*>(pbase + NP * 256 + off) = __float2bfloat16(p - __bfloat162float(hi));
+        *reinterpret_cast<__nv_bfloat16*>(pbase + NP * 128 + off) = __float2bfloat16(p - __bfloat162float(hi));
       }
       if (b > 0 && grew[0]) {
         // s_full of this block was committed after the products of the previous one: O is at rest
-        for (int m = 0; m < ns; ++m) {
+        for (int m = 0; m < 2 * ns; ++m) {
           uint32_t o[CPT];
           __syncwarp();
           lt_ld<CPT>(t_s + NP * (1 + m), o);
@@ -297,21 +296,23 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
     if (ok) {
       tc_fence_after();
       for (int m = 0; m < ns; ++m) {
-        uint32_t o[CPT];
+        uint32_t o[CPT], lo[CPT];
         __syncwarp();
-        lt_ld<CPT>(t_s + NP * (1 + m), o);
+        lt_ld<CPT>(t_s + NP * (1 + 2 * m), o);
+        lt_ld<CPT>(t_s + NP * (2 + 2 * m), lo);
         tmem_ld_wait();
         const int r = m * 128 + kin;
 #pragma unroll
         for (int j = 0; j < CPT; ++j) {
           const int hr = half * CPT + j;
           if (hr >= nh || r >= R) continue;
+          const float ov = __uint_as_float(o[j]) + __uint_as_float(lo[j]);
           const float l = lred[hr] + lred[NP + hr] + lred[2 * NP + hr] + lred[3 * NP + hr];
           const long long row = t * c.heads + h0 + hr;
           if (a.splits == 1) {
-            a.out[row * R + r] = __float2bfloat16(__uint_as_float(o[j]) / l);
+            a.out[row * R + r] = __float2bfloat16(ov / l);
           } else {
-            a.part[(row * a.splits + split) * R + r] = __uint_as_float(o[j]);
+            a.part[(row * a.splits + split) * R + r] = ov;
             if (r == 0) {
               a.ml[(row * a.splits + split) * 2] = stat[hr];
               a.ml[(row * a.splits + split) * 2 + 1] = l;

@@ -17,42 +17,62 @@
 namespace cgk {
 namespace {
 
-template <typename TI, typename T>
-__global__ void latent_norm_append_kernel(const TI* __restrict__ in, long long ld, const float* __restrict__ wq, const float* __restrict__ wc,
-                                          int q_rank, int R, float eps, T* __restrict__ cq, T* __restrict__ c_out, T* __restrict__ pages,
-                                          const int* __restrict__ slot, const int* __restrict__ pos, const int* __restrict__ page_table,
-                                          int slots, int max_pages, int page_size, int n_pages) {
-  __shared__ float red[33];
+// One CTA per token; the row stays in shared memory between the sums of squares and the scaling.
+template <typename TI, typename T, int V>
+__global__ void __launch_bounds__(256)
+latent_norm_append_kernel(const TI* __restrict__ in, long long ld, const float* __restrict__ wq, const float* __restrict__ wc, int q_rank, int R,
+                          float eps, T* __restrict__ cq, T* __restrict__ c_out, T* __restrict__ pages, const int* __restrict__ slot,
+                          const int* __restrict__ pos, const int* __restrict__ page_table, int slots, int max_pages, int page_size, int n_pages) {
+  extern __shared__ float row_buf[];
+  __shared__ float red[64];
   const long long t = blockIdx.x;
-  const TI* row = in + t * ld;
-  float sq = 0.0f, sc = 0.0f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = ld1(row + i); sq = fmaf(v, v, sq); }
-  for (int i = threadIdx.x; i < R; i += blockDim.x) { const float v = ld1(row + q_rank + i); sc = fmaf(v, v, sc); }
-  sq = block_sum(sq, red);
-  sc = block_sum(sc, red);
-  const float rq = 1.0f / sqrtf(sq / q_rank + eps), rc = 1.0f / sqrtf(sc / R + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) st1(cq + t * q_rank + i, ld1(row + i) * rq * wq[i]);
+  const int n = q_rank + R, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int p = (int)CGK_IDX(pos[t], (long long)max_pages * page_size), s = (int)CGK_IDX(slot[t], slots);
   const long long page = CGK_IDX(page_table[(long long)s * max_pages + p / page_size], n_pages);
+  float sq = 0.0f, sc = 0.0f;
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {        // q_rank is a multiple of V: no vector straddles
+    float v[V], ss = 0.0f;
+    ldv<V>(in + t * ld + i, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) { ss = fmaf(v[j], v[j], ss); row_buf[i + j] = v[j]; }
+    if (i < q_rank) sq += ss; else sc += ss;
+  }
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
+  if (lane == 0) { red[warp] = sq; red[32 + warp] = sc; }
+  __syncthreads();
+  sq = sc = 0.0f;
+  for (int w = 0; w < nw; ++w) { sq += red[w]; sc += red[32 + w]; }
+  const float rq = 1.0f / sqrtf(sq / q_rank + eps), rc = 1.0f / sqrtf(sc / R + eps);
   T* dst = pages + (page * page_size + p % page_size) * R;
-  for (int i = threadIdx.x; i < R; i += blockDim.x) {
-    const float v = ld1(row + q_rank + i) * rc * wc[i];
-    st1(dst + i, v);
-    if (c_out) st1(c_out + t * R + i, v);
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+    float v[V], w[V];
+    const bool isq = i < q_rank;
+    ldv<V>(isq ? wq + i : wc + i - q_rank, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] = row_buf[i + j] * (isq ? rq : rc) * w[j];
+    if (isq) {
+      stv<V>(cq + t * q_rank + i, v);
+    } else {
+      stv<V>(dst + i - q_rank, v);
+      if (c_out) stv<V>(c_out + t * R + i - q_rank, v);
+    }
   }
 }
 
+// One warp per row.
 template <typename T>
-__global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __restrict__ table_row, T* __restrict__ out, int R, int page_size,
+__global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __restrict__ table_row, T* __restrict__ out, int len, int R, int page_size,
                                      int max_pages, int n_pages) {
-  const int p = blockIdx.x;
+  const int p = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (p >= len) return;
   const long long page = CGK_IDX(table_row[CGK_IDX(p / page_size, max_pages)], n_pages);
   const T* src = pages + (page * page_size + p % page_size) * R;
   T* dst = out + (long long)p * R;
-  if (R % 8 == 0 && sizeof(T) == 2) {
-    for (int i = threadIdx.x; i < R / 8; i += blockDim.x) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+  if ((R * (int)sizeof(T)) % 16 == 0) {
+    for (int i = lane; i < R * (int)sizeof(T) / 16; i += 32) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
   } else {
-    for (int i = threadIdx.x; i < R; i += blockDim.x) dst[i] = src[i];
+    for (int i = lane; i < R; i += 32) dst[i] = src[i];
   }
 }
 
@@ -118,24 +138,28 @@ latent_attention_kernel(const LatentDev c, const T* __restrict__ q, T* __restric
   }
 }
 
-// Partials of key ranges -> result: out[row][r] = sum_s acc[row][s][r] 2^(m_s - m) / sum_s l_s 2^(m_s - m)
+// Partials of up to 32 key ranges -> result: out[row][r] = sum_s acc[row][s][r] 2^(m_s - m) / sum_s l_s 2^(m_s - m)
 __global__ void latent_merge_kernel(const float* __restrict__ part, const float* __restrict__ ml, __nv_bfloat16* __restrict__ out, int splits, int R) {
+  __shared__ float weight[32];
   const long long row = blockIdx.x;
-  float m = -INFINITY;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[(row * splits + s) * 2]);
-  float l = 0.0f;
-  for (int s = 0; s < splits; ++s) {
-    const float ms = ml[(row * splits + s) * 2];
-    if (ms > -INFINITY) l = fmaf(ml[(row * splits + s) * 2 + 1], exp2f(ms - m), l);
+  const int lane = threadIdx.x & 31;
+  if (threadIdx.x < 32) {
+    const float2 v = lane < splits ? reinterpret_cast<const float2*>(ml)[row * splits + lane] : make_float2(-INFINITY, 0.0f);
+    const float m = warp_max(v.x);
+    const float f = v.x > -INFINITY ? exp2f(v.x - m) : 0.0f;
+    weight[lane] = f / warp_sum(v.y * f);
   }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  __syncthreads();
+  const float* p = part + row * splits * R;
   for (int r = threadIdx.x; r < R; r += blockDim.x) {
     float v = 0.0f;
+#pragma unroll 8
     for (int s = 0; s < splits; ++s) {
-      const float ms = ml[(row * splits + s) * 2];
-      if (ms > -INFINITY) v = fmaf(part[(row * splits + s) * R + r], exp2f(ms - m), v);
+      const float w = weight[s];
+      // a range without keys wrote no sums
+      if (w > 0.0f) v = fmaf(p[(long long)s * R + r], w, v);
     }
-    out[row * R + r] = __float2bfloat16(v * inv);
+    out[row * R + r] = __float2bfloat16(v);
   }
 }
 
@@ -184,10 +208,22 @@ CGK_API int cgk_latent_norm_append(const cgk_latent_args* pa, const void* in, in
   if (rows == 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   typedef __nv_bfloat16 bf;
+  const int n = q_rank + d.R, smem = n * 4;
+  CGK_REQUIRE(smem <= 48 * 1024, "cgk_latent_norm_append: rows of %d elements are too long", n);
+  auto al = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
+  const bool vec = q_rank % 4 == 0 && d.R % 4 == 0 && ld % 4 == 0 && al(in) && al(wq) && al(wc) && al(cq) && al(c_out) && al(d.pages);
+  const int nt = n >= 2048 ? 256 : 128;
 #define CGK_LNA(TI, T)                                                                                                              \
-  latent_norm_append_kernel<TI, T><<<rows, 128, 0, st>>>((const TI*)in, ld, (const float*)wq, (const float*)wc, q_rank, d.R, eps,  \
-                                                        (T*)cq, (T*)c_out, (T*)d.pages, d.slot, d.pos, d.page_table, d.slots,     \
-                                                        d.max_pages, d.page_size, d.n_pages)
+  do {                                                                                                                             \
+    if (vec)                                                                                                                       \
+      latent_norm_append_kernel<TI, T, 4><<<rows, nt, smem, st>>>((const TI*)in, ld, (const float*)wq, (const float*)wc, q_rank,   \
+                                                                  d.R, eps, (T*)cq, (T*)c_out, (T*)d.pages, d.slot, d.pos,         \
+                                                                  d.page_table, d.slots, d.max_pages, d.page_size, d.n_pages);     \
+    else                                                                                                                           \
+      latent_norm_append_kernel<TI, T, 1><<<rows, nt, smem, st>>>((const TI*)in, ld, (const float*)wq, (const float*)wc, q_rank,   \
+                                                                  d.R, eps, (T*)cq, (T*)c_out, (T*)d.pages, d.slot, d.pos,         \
+                                                                  d.page_table, d.slots, d.max_pages, d.page_size, d.n_pages);     \
+  } while (0)
   if (pa->fp32) {
     CGK_REQUIRE(in_fp32, "cgk_latent_norm_append: the fp32 form takes fp32 inputs");
     CGK_LNA(float, float);
@@ -207,8 +243,8 @@ CGK_API int cgk_latent_gather(const cgk_latent_args* pa, int slot, int len, void
   if (len == 0) return 0;
   const int* row = (const int*)pa->page_table + (long long)slot * pa->max_pages;
   cudaStream_t st = (cudaStream_t)stream;
-  if (pa->fp32) latent_gather_kernel<float><<<len, 64, 0, st>>>((const float*)pa->pages, row, (float*)out, pa->R, pa->page_size, pa->max_pages, pa->n_pages);
-  else latent_gather_kernel<__nv_bfloat16><<<len, 64, 0, st>>>((const __nv_bfloat16*)pa->pages, row, (__nv_bfloat16*)out, pa->R, pa->page_size, pa->max_pages, pa->n_pages);
+  if (pa->fp32) latent_gather_kernel<float><<<(len + 3) / 4, 128, 0, st>>>((const float*)pa->pages, row, (float*)out, len, pa->R, pa->page_size, pa->max_pages, pa->n_pages);
+  else latent_gather_kernel<__nv_bfloat16><<<(len + 3) / 4, 128, 0, st>>>((const __nv_bfloat16*)pa->pages, row, (__nv_bfloat16*)out, len, pa->R, pa->page_size, pa->max_pages, pa->n_pages);
   CGK_LAUNCH_CHECK();
   return 0;
 }
@@ -228,7 +264,7 @@ CGK_API int cgk_latent_attention(const cgk_latent_args* pa, const void* q, void*
   if (rows == 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   if (!pa->fp32 && !force_simt && latent_tc_ok(d.R, d.page_size, d.heads)) {
-    CGK_REQUIRE(splits >= 1 && (splits == 1 || scratch), "cgk_latent_attention: key splits need scratch space");
+    CGK_REQUIRE(splits >= 1 && splits <= 32 && (splits == 1 || scratch), "cgk_latent_attention: up to 32 key ranges, with scratch space");
     return launch_latent_tc(d, (const __nv_bfloat16*)q, (__nv_bfloat16*)out, rows, splits, (float*)scratch, st);
   }
   CGK_REQUIRE(d.R <= 1024, "cgk_latent_attention: latents of %d elements are longer than the 1024 supported", d.R);

@@ -293,6 +293,11 @@ int cgk_rms_rows(const void* x, const void* rows, int n_out, int n_rows, const v
 int cgk_gemm_f32(const void* A, const void* B, void* C, int M, int N, int K, int batch, long long lda, long long ldb, long long ldc,
                  long long sA, long long sB, long long sC, int b_mn, void* stream);
 
+/* Products with up to 8 rows (decoding), bf16 operands, fp32 sums: out[b, m, n] = sum_k x[b, m, k] W[b, n, k].
+ * mode 0: plain; 1: gated, W holds N gate rows then N up rows and out = silu(gate) * up (batch 1); 2: W stored [K, N]. */
+int cgk_skinny_gemm(const void* x, long long ldx, long long sx, const void* w, long long ldw, long long sw, void* out, long long ldo,
+                    long long so, int out_fp32, int M, int N, int K, int batch, int mode, void* stream);
+
 /* ---- Latent attention (csrc/kernels/latent_kv.cu, latent_attn_tc.cu) ---- */
 /* One layer's paged cache of latents, pages[n_pages][page_size][R] in bf16 (fp32 with `fp32`), and the query
  * tokens of a call: token t belongs to the sequence in slot[t] and stands at pos[t]. */

@@ -84,6 +84,32 @@ def test_fp32_product_is_not_a_reduced_precision_one(b_mn):
     assert torch.allclose(out.cpu().double(), torch.einsum("nhk,hkr->nhr", a.view(6, 4, 10).cpu().double(), w.cpu().double()), atol=1e-4)
 
 
+@pytest.mark.parametrize("M", [1, 2, 3, 5, 8, 9])
+@pytest.mark.parametrize("N,K", [(3, 8), (100, 264), (2500, 520), (12001, 64), (40, 4104)])
+def test_products_with_few_rows(M, N, K):
+    from cogito_b200.ops.linear import gated_linear, linear
+    a, w = rand(M, K, seed=1, dtype=BF), rand(N, K, seed=2, dtype=BF, scale=K ** -0.5)
+    want = a.double() @ w.double().T
+    for dt, tol in ((F32, 2e-5), (BF, 1e-2)):
+        got = linear(a.to(DEV), w.to(DEV), out_dtype=dt)
+        assert got.dtype == dt and float((got.cpu().double() - want).abs().max()) < tol * max(1.0, float(want.abs().max()))
+    w2 = rand(2 * N, K, seed=3, dtype=BF, scale=K ** -0.5)
+    want = plain.silu(a.double() @ w2[:N].double().T) * (a.double() @ w2[N:].double().T)
+    got = gated_linear(a.to(DEV), w2.to(DEV))
+    assert float((got.cpu().double() - want).abs().max()) < 2e-2 * max(1.0, float(want.abs().max()))
+    # heads interleaved in the rows, both storage orders
+    H, D, R = 3, 40, 136
+    x, wk, wv = rand(M, H * D, seed=4, dtype=BF), rand(H, D, R, seed=5, dtype=BF), rand(H, D, R, seed=6, dtype=BF)
+    xh, up = x.to(DEV).view(M, H, D).transpose(0, 1), torch.empty(M, H, R, dtype=BF, device=DEV)
+    linear(xh, wk.to(DEV), w_mn=True, out=up.transpose(0, 1))
+    want = torch.einsum("mhd,hdr->mhr", x.view(M, H, D).double(), wk.double())
+    assert float((up.cpu().double() - want).abs().max()) < 1e-2 * float(want.abs().max())
+    down = torch.empty(M, H * D, dtype=BF, device=DEV)
+    linear(up.transpose(0, 1), wv.to(DEV), out=down.view(M, H, D).transpose(0, 1))
+    want = torch.einsum("mhr,hdr->mhd", up.cpu().double(), wv.double()).reshape(M, H * D)
+    assert float((down.cpu().double() - want).abs().max()) < 1e-2 * float(want.abs().max())
+
+
 def _latents(R, dtype, lengths, page_size=64, seed=0, extra_pages=3):
     """A cache whose sequences own shuffled pages, filled with the given numbers of random latents."""
     g = torch.Generator().manual_seed(seed)
