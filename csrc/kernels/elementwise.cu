@@ -14,6 +14,7 @@
 #include "../../include/cogito_kernels.h"
 #include "host_common.h"
 #include "sm100.cuh"
+#include "swiglu_rows.cuh"
 
 namespace cgk {
 
@@ -381,6 +382,10 @@ __global__ void swiglu_fwd_kernel(const T* __restrict__ x, T* __restrict__ y, lo
     stf<T>(y, i, silu_f(g) * v);
   }
 }
+__global__ void __launch_bounds__(256)
+swiglu_fwd_rows_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ y, long long rows, int H) {
+  swiglu_rows_bf16(x, y, rows, H);
+}
 template <typename T>
 __global__ void swiglu_bwd_kernel(const T* __restrict__ x, const T* __restrict__ dy,
                                   T* __restrict__ dx, long long rows, int H) {
@@ -724,6 +729,8 @@ CGK_API int cgk_swiglu_forward(int dtype, const void* x, void* y, long long rows
   CGK_REQUIRE(x && y && H > 0, "cgk_swiglu_forward: bad argument");
   if (rows == 0) return 0;
   if (dtype == 0) swiglu_fwd_kernel<float><<<ew_grid(rows * H), 256, 0, ST(stream)>>>((const float*)x, (float*)y, rows, H);
+  else if (H % 8 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0)
+    swiglu_fwd_rows_kernel<<<swiglu_rows_grid(rows), swiglu_rows_threads(H), 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
   else swiglu_fwd_kernel<__nv_bfloat16><<<ew_grid(rows * H), 256, 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
   CGK_LAUNCH_CHECK();
   return 0;

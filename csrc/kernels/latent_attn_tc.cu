@@ -71,8 +71,8 @@ struct LtSmem {
   static __host__ __device__ uint32_t off_t(int slots, int ns) { return off_q(slots) + ns * NP * 256; }
   static __host__ __device__ uint32_t off_stat(int slots, int ns) { return off_t(slots, ns) + T_BYTES; }          // float [3][NP]
   static __host__ __device__ uint32_t off_lred(int slots, int ns) { return off_stat(slots, ns) + 3 * NP * 4; }    // float [4][NP]
-  static __host__ __device__ uint32_t off_bar(int slots, int ns) { return off_lred(slots, ns) + 4 * NP * 4; }     // full, empty, s_full, p_ready, o_full
-  static __host__ __device__ uint32_t off_misc(int slots, int ns) { return off_bar(slots, ns) + (2 * LT_MAX_SLOTS + 3) * 8 + 8; }
+  static __host__ __device__ uint32_t off_bar(int slots, int ns) { return off_lred(slots, ns) + 4 * NP * 4; }     // full, empty, s_full, p_ready, o_full, q_full
+  static __host__ __device__ uint32_t off_misc(int slots, int ns) { return off_bar(slots, ns) + (2 * LT_MAX_SLOTS + 4) * 8; }
   static __host__ __device__ uint32_t total(int slots, int ns) { return off_misc(slots, ns) + 32 + 1024; }
 };
 
@@ -109,7 +109,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
   float* lred = reinterpret_cast<float*>(sm + S::off_lred(slots, ns));
   auto full_bar = [&](int s) { return sb + o_bar + 8u * s; };
   auto empty_bar = [&](int s) { return sb + o_bar + 8u * (LT_MAX_SLOTS + s); };
-  const uint32_t s_full = sb + o_bar + 8u * (2 * LT_MAX_SLOTS), p_ready = s_full + 8, o_full = s_full + 16;
+  const uint32_t s_full = sb + o_bar + 8u * (2 * LT_MAX_SLOTS), p_ready = s_full + 8, o_full = s_full + 16, q_full = s_full + 24;
   volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(sm + o_misc);
   volatile int* dead = reinterpret_cast<volatile int*>(sm + o_misc + 4);
   volatile int* go = reinterpret_cast<volatile int*>(sm + o_misc + 8);
@@ -122,6 +122,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
     mbar_init(s_full, 1);
     mbar_init(p_ready, 8);
     mbar_init(o_full, 1);
+    mbar_init(q_full, 8);
     *dead = 0;
     mbar_fence_init();
   }
@@ -129,15 +130,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
     tmem_alloc(sb + o_misc, cols);
     tmem_relinquish();
   }
-  // queries -> K-major operand tiles [NP][64] per 64 latent columns, zeros beyond the heads and beyond R
-  for (int i = tid; i < NP * ns * 16; i += LT_THREADS) {
-    const int r = i / (ns * 16), ch = i % (ns * 16), col = ch * 8;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < nh && col < R) v = *reinterpret_cast<const uint4*>(a.q + (t * c.heads + h0 + r) * R + col);
-    *reinterpret_cast<uint4*>(sm + o_q + (ch >> 3) * (NP * 128) + sw128_offset(r, ch & 7)) = v;
-  }
   if (tid < NP) stat[tid] = -INFINITY;
-  fence_proxy_async_smem();
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -173,7 +166,8 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
   } else if (warp == 9) {
     if (lane == 0) {
       const uint32_t id_s = make_idesc_bf16(128, NP, 0, 0), id_o = make_idesc_bf16(128, 2 * NP, 1, 0);
-      bool ok = true;
+      bool ok = mbar_wait(q_full, 0, dead, a.status, 712);
+      tc_fence_after();
       for (int b = 0; b < nblk && ok; ++b) {
         for (int m = 0; m < ns; ++m) {
           const int it = b * ns + m, s = it % slots;
@@ -201,6 +195,17 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
       }
     }
   } else {
+    // queries -> K-major operand tiles [NP][64] per 64 latent columns, zeros beyond the heads and beyond R; the
+    // first key block is already on its way
+#pragma unroll 4
+    for (int i = tid; i < ns * NP * 16; i += LT_SOFT) {
+      const int ch = i & 15, r = (i >> 4) % NP, m = (i >> 4) / NP, col = m * 128 + ch * 8;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (r < nh && col < R) v = *reinterpret_cast<const uint4*>(a.q + (t * c.heads + h0 + r) * R + col);
+      *reinterpret_cast<uint4*>(sm + o_q + (m * 2 + (ch >> 3)) * (NP * 128) + sw128_offset(r, ch & 7)) = v;
+    }
+    fence_proxy_async_smem();
+    mbar_arrive_warp(q_full);
     const int quad = warp & 3, half = warp >> 2;
     const uint32_t t_s = tmem + ((uint32_t)(quad * 32) << 16) + half * CPT;
     const int kin = quad * 32 + lane;

@@ -151,16 +151,15 @@ __global__ void latent_merge_kernel(const float* __restrict__ part, const float*
   }
   __syncthreads();
   const float* p = part + row * splits * R;
-  for (int r = threadIdx.x; r < R; r += blockDim.x) {
-    float v = 0.0f;
-#pragma unroll 8
-    for (int s = 0; s < splits; ++s) {
-      const float w = weight[s];
-      // a range without keys wrote no sums
-      if (w > 0.0f) v = fmaf(p[(long long)s * R + r], w, v);
-    }
-    out[row * R + r] = __float2bfloat16(v);
+  const int r = blockIdx.y * blockDim.x + threadIdx.x;
+  if (r >= R) return;
+  float v = 0.0f;
+#pragma unroll 16
+  for (int s = 0; s < splits; ++s) {
+    const float e = p[(long long)s * R + r], w = weight[s];
+    v += w > 0.0f ? w * e : 0.0f;                    // a range without keys wrote no sums: its memory is not looked at
   }
+  out[row * R + r] = __float2bfloat16(v);
 }
 
 template <typename T, int NR>
@@ -191,7 +190,7 @@ int fill_latent(const cgk_latent_args& a, LatentDev* d) {
 }  // namespace
 
 cudaError_t launch_latent_merge(const float* part, const float* ml, __nv_bfloat16* out, int rows, int splits, int R, cudaStream_t st) {
-  latent_merge_kernel<<<rows, R <= 128 ? 64 : 128, 0, st>>>(part, ml, out, splits, R);
+  latent_merge_kernel<<<dim3(rows, (R + 127) / 128), 128, 0, st>>>(part, ml, out, splits, R);
   return cudaGetLastError();
 }
 

@@ -11,6 +11,7 @@
 #include "../../include/cogito_kernels.h"
 #include "host_common.h"
 #include "sm100.cuh"
+#include "swiglu_rows.cuh"
 #include "typed_io.cuh"
 
 namespace cgk {
@@ -155,22 +156,9 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ h, const int
 }
 
 // act[row][f] = silu(gu[row][f]) * gu[row][F + f] over the rows in use (*tiles * 128)
-__global__ void swiglu_tiles_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act, const int* __restrict__ tiles, int F) {
-  const long long n = (long long)*tiles * 128 * (F / 8);
-  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    const long long row = i / (F / 8);
-    const int f = (int)(i % (F / 8)) * 8;
-    const uint4 g = *reinterpret_cast<const uint4*>(gu + row * 2 * F + f);
-    const uint4 u = *reinterpret_cast<const uint4*>(gu + row * 2 * F + F + f);
-    const uint32_t gw[4] = {g.x, g.y, g.z, g.w}, uw[4] = {u.x, u.y, u.z, u.w};
-    uint32_t o[4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float2 a = unpack_bf16x2(gw[j]), b = unpack_bf16x2(uw[j]);
-      o[j] = pack_bf16x2(silu_f(a.x) * b.x, silu_f(a.y) * b.y);
-    }
-    *reinterpret_cast<uint4*>(act + row * F + f) = make_uint4(o[0], o[1], o[2], o[3]);
-  }
+__global__ void __launch_bounds__(256)
+swiglu_tiles_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act, const int* __restrict__ tiles, int F) {
+  swiglu_rows_bf16(gu, act, (long long)*tiles * 128, F);
 }
 
 template <typename T, int V>
@@ -261,9 +249,7 @@ CGK_API int cgk_moe_gather(const void* h, const void* idx, int pairs, int top, i
 CGK_API int cgk_swiglu_tiles(const void* gu, void* act, const void* tiles, int F, int max_tiles, void* stream) {
   CGK_REQUIRE(gu && act && tiles && F % 8 == 0 && F > 0, "cgk_swiglu_tiles: rows must be multiples of 8 elements");
   if (max_tiles == 0) return 0;
-  const long long work = (long long)max_tiles * 128 * (F / 8);
-  const int blocks = (int)((work + 255) / 256 < 148 * 8 ? (work + 255) / 256 : 148 * 8);
-  swiglu_tiles_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act, (const int*)tiles, F);
+  swiglu_tiles_kernel<<<swiglu_rows_grid((long long)max_tiles * 128), swiglu_rows_threads(F), 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act, (const int*)tiles, F);
   CGK_LAUNCH_CHECK();
   return 0;
 }

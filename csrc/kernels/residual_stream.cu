@@ -94,6 +94,100 @@ __global__ void stream_update_kernel(const UpdateDev a) {
   }
 }
 
+// The same update with the row in registers: 8 elements per thread and step, the stream requested together with
+// the sublayer's result so that one round trip covers both.
+template <typename T>
+__device__ __forceinline__ void ld8(const T* p, float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    const uint4 t = *reinterpret_cast<const uint4*>(p);
+    float2 f;
+    f = unpack_bf16x2(t.x); v[0] = f.x; v[1] = f.y;
+    f = unpack_bf16x2(t.y); v[2] = f.x; v[3] = f.y;
+    f = unpack_bf16x2(t.z); v[4] = f.x; v[5] = f.y;
+    f = unpack_bf16x2(t.w); v[6] = f.x; v[7] = f.y;
+  } else {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+}
+template <typename T>
+__device__ __forceinline__ void st8(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  } else {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+template <typename TY, typename TP, typename TH, int ITER>
+__global__ void __launch_bounds__(512)
+stream_update_regs_kernel(const UpdateDev a) {
+  __shared__ float red[16];
+  const long long t = blockIdx.x;
+  const TY* y = reinterpret_cast<const TY*>(a.y);
+  const TP* pairs = reinterpret_cast<const TP*>(a.pairs);
+  float* x = a.x + t * a.D;
+  float v[ITER][8], xv[ITER][8], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.D) {
+      ld8(x + c, xv[i]);
+      if (y) {
+        ld8(y + t * a.ldy + c, v[i]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[i][j] = 0.0f;
+      }
+    }
+  }
+#pragma unroll 4
+  for (int k = 0; k < a.top; ++k) {
+    const int r = a.row_of[t * a.top + k];
+    const float wk = a.weight[t * a.top + k];
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 8;
+      if (c < a.D) {
+        if (r >= 0) {
+          float e[8];
+          ld8(pairs + CGK_IDX(r, a.pair_rows) * a.ldp + c, e);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[i][j] = fmaf(wk, e[j], v[i][j]);
+        } else {                                       // an expert whose output is its input
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[i][j] = fmaf(wk, xv[i][j], v[i][j]);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < ITER; ++i)
+    if ((i * blockDim.x + threadIdx.x) * 8 < a.D) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[i][j], v[i][j], ss);
+    }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.0f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += red[w];
+  const float rstd = 1.0f / sqrtf(ss / a.D + a.eps);
+  TH* h = reinterpret_cast<TH*>(a.h) + t * a.D;
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.D) {
+      float wv[8];
+      ld8(a.w + c, wv);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) xv[i][j] += v[i][j] * rstd * wv[j];
+      st8(x + c, xv[i]);
+      st8(h + c, xv[i]);
+    }
+  }
+}
+
 template <typename TO>
 __global__ void rms_rows_kernel(const float* __restrict__ x, const long long* __restrict__ rows, int n_rows, const float* __restrict__ w,
                                 TO* __restrict__ out, int D, float eps) {
@@ -112,6 +206,16 @@ int row_threads(int n) { return n <= 64 ? 64 : (n >= 512 ? 512 : (n + 31) / 32 *
 
 template <typename TY, typename TP, typename TH>
 int launch_update(const UpdateDev& d, int rows, bool vec, cudaStream_t st) {
+  auto a16 = [](const void* p, long long row_bytes) { return !p || ((((uintptr_t)p) & 15) == 0 && row_bytes % 16 == 0); };
+  if (d.D % 8 == 0 && d.D <= 512 * 8 * 4 && a16(d.y, d.ldy * sizeof(TY)) && a16(d.pairs, d.ldp * sizeof(TP)) && a16(d.x, 0) && a16(d.w, 0) &&
+      a16(d.h, 0)) {
+    const int vecs = d.D / 8, iter = vecs <= 512 ? 1 : (vecs <= 1024 ? 2 : 4), nt = ((vecs + iter - 1) / iter + 31) / 32 * 32;
+    if (iter == 1) stream_update_regs_kernel<TY, TP, TH, 1><<<rows, nt, 0, st>>>(d);
+    else if (iter == 2) stream_update_regs_kernel<TY, TP, TH, 2><<<rows, nt, 0, st>>>(d);
+    else stream_update_regs_kernel<TY, TP, TH, 4><<<rows, nt, 0, st>>>(d);
+    CGK_LAUNCH_CHECK();
+    return 0;
+  }
   const int smem = d.D * 4;
   const int nt = row_threads(vec ? d.D / 4 : d.D);
   if (vec) {
