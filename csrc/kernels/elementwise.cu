@@ -730,7 +730,7 @@ CGK_API int cgk_swiglu_forward(int dtype, const void* x, void* y, long long rows
   if (rows == 0) return 0;
   if (dtype == 0) swiglu_fwd_kernel<float><<<ew_grid(rows * H), 256, 0, ST(stream)>>>((const float*)x, (float*)y, rows, H);
   else if (H % 8 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0)
-    swiglu_fwd_rows_kernel<<<swiglu_rows_grid(rows), swiglu_rows_threads(H), 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
+    swiglu_fwd_rows_kernel<<<swiglu_rows_grid(rows, H), swiglu_rows_threads(H), 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
   else swiglu_fwd_kernel<__nv_bfloat16><<<ew_grid(rows * H), 256, 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
   CGK_LAUNCH_CHECK();
   return 0;

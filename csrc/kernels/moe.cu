@@ -249,7 +249,7 @@ CGK_API int cgk_moe_gather(const void* h, const void* idx, int pairs, int top, i
 CGK_API int cgk_swiglu_tiles(const void* gu, void* act, const void* tiles, int F, int max_tiles, void* stream) {
   CGK_REQUIRE(gu && act && tiles && F % 8 == 0 && F > 0, "cgk_swiglu_tiles: rows must be multiples of 8 elements");
   if (max_tiles == 0) return 0;
-  swiglu_tiles_kernel<<<swiglu_rows_grid((long long)max_tiles * 128), swiglu_rows_threads(F), 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act, (const int*)tiles, F);
+  swiglu_tiles_kernel<<<swiglu_rows_grid((long long)max_tiles * 128, F), swiglu_rows_threads(F), 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act, (const int*)tiles, F);
   CGK_LAUNCH_CHECK();
   return 0;
 }

@@ -1,5 +1,5 @@
 // silu(gate) * up over bf16 rows [gate | up] of 2 F elements, F a multiple of 8: four rows at a time per CTA, so every
-// thread keeps eight 16-byte loads in flight.
+// thread keeps eight 16-byte loads in flight.  blockIdx.y picks a range of columns (few long rows still fill the GPU).
 #pragma once
 #include "sm100.cuh"
 
@@ -9,7 +9,8 @@ constexpr int SWIGLU_ROWS = 4;
 
 __device__ __forceinline__ void swiglu_rows_bf16(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act, long long rows, int F) {
   for (long long row0 = (long long)blockIdx.x * SWIGLU_ROWS; row0 < rows; row0 += (long long)gridDim.x * SWIGLU_ROWS) {
-    for (int f = threadIdx.x * 8; f < F; f += blockDim.x * 8) {
+    const int f = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+    if (f < F) {
       uint4 g[SWIGLU_ROWS], u[SWIGLU_ROWS];
 #pragma unroll
       for (int j = 0; j < SWIGLU_ROWS; ++j) {
@@ -35,9 +36,10 @@ __device__ __forceinline__ void swiglu_rows_bf16(const __nv_bfloat16* __restrict
 }
 
 inline int swiglu_rows_threads(int F) { return F / 8 >= 256 ? 256 : (F / 8 + 31) / 32 * 32; }
-inline int swiglu_rows_grid(long long rows) {
-  const long long n = (rows + SWIGLU_ROWS - 1) / SWIGLU_ROWS;
-  return (int)(n < 148 * 16 ? (n < 1 ? 1 : n) : 148 * 16);
+inline dim3 swiglu_rows_grid(long long rows, int F) {
+  const int nt = swiglu_rows_threads(F), cols = (F / 8 + nt - 1) / nt;
+  long long n = (rows + SWIGLU_ROWS - 1) / SWIGLU_ROWS, cap = 148 * 16 / (cols < 16 ? cols : 16);
+  return dim3((unsigned)(n < 1 ? 1 : (n < cap ? n : cap)), cols);
 }
 
 }  // namespace cgk
