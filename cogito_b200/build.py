@@ -104,10 +104,10 @@ SERVE_SOURCES = ("elementwise", "flash_fwd", "gemm_f32", "gemm_tcgen05", "host_c
                  "kv_attn_tc", "residual_stream", "serving", "skinny_gemm")
 
 
-def build_serving_kernels(verbose: bool = False) -> Path:
+def build_serving_kernels(verbose: bool = False, out: Path | None = None) -> Path:
     """``libcogito_kernels_serve.so``: the subset of the kernel library in SERVE_SOURCES."""
     srcs = [ROOT / "csrc" / "kernels" / f"{name}.cu" for name in SERVE_SOURCES]
-    out = LIB_DIR / "libcogito_kernels_serve.so"
+    out = out or LIB_DIR / "libcogito_kernels_serve.so"
     nvcc = _nvcc()
     _build(srcs, _kernel_headers(), out, [nvcc] + NVCC_FLAGS + ["-I", str(ROOT / "include")],
            [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC", "-cudart", "shared"], "kernels", verbose)

@@ -44,8 +44,10 @@ def _fns():
     global _declared
     L = _lib.lib()
     if not _declared:
-        L.cgk_flash_forward.argtypes = [POINTER(FlashArgs), c_void_p]
-        L.cgk_flash_backward.argtypes = [POINTER(FlashArgs), c_void_p]
+        for name in ("cgk_flash_forward", "cgk_flash_backward"):
+            fn = getattr(L, name, None)                 # a library built for serving has no backward kernels
+            if fn is not None:
+                fn.argtypes = [POINTER(FlashArgs), c_void_p]
         _declared = True
     return L
 

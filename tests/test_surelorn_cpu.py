@@ -273,3 +273,29 @@ def test_trace_replay_and_command_line(tmp_path):
     out = main(base + [f"generate.draft_path={folder}", "generate.batch=2", "generate.prompt_len=6"])
     seqs = json.loads((tmp_path / "o.json").read_text())
     assert all(s[6:11] == _greedy(d, t, s[:6], 5) for s in seqs)
+
+
+def test_the_serving_subset_of_the_kernels_has_what_the_engine_calls(tmp_path):
+    """A checkout that only serves compiles part of the library: it must load, and every function that the modules
+    on the serving path name must be in it."""
+    import ctypes
+    import re
+    import subprocess
+    import sys
+    from pathlib import Path
+
+    from cogito_b200 import build
+    root = Path(__file__).resolve().parent.parent
+    if not all((build.BUILD_DIR / "kernels" / f"{n}.o").exists() for n in build.SERVE_SOURCES):
+        pytest.skip("kernel objects have not been compiled here")
+    so = build.build_serving_kernels(out=tmp_path / "serve.so")
+    lib = ctypes.CDLL(str(so))
+    named = set()
+    for f in ("ops/stream.py", "ops/moe.py", "ops/linear.py", "ops/gemm.py", "serve/kv_cache.py", "serve/sampling.py"):
+        named |= set(re.findall(r"\.(cgk_\w+)\(", (root / "cogito_b200" / f).read_text()))
+    assert len(named) > 15 and not [n for n in named if not hasattr(lib, n)]
+    # the bindings accept a library without the training kernels
+    code = ("import sys; sys.path.insert(0, sys.argv[1]); from pathlib import Path; from cogito_b200.ops import _lib, attention; "
+            "_lib._LIB_PATH = Path(sys.argv[2]); L = attention._fns(); print(L.cgk_version(), bool(L.cgk_flash_forward.argtypes))")
+    r = subprocess.run([sys.executable, "-c", code, str(root), str(so)], capture_output=True, text=True)
+    assert r.returncode == 0 and r.stdout.split()[1] == "True", r.stderr
