@@ -47,7 +47,7 @@ def test_plain_router_keeps_groups_by_their_best_choice_score_and_weighs_without
     got = plain.choose(logits, corr, {"groups": {"count": 3, "keep": 2}, "top": 3})
     assert [i for i, _ in got] == [4, 2, 3]
     assert [round(float(v), 6) for _, v in got] == [round(v / 0.41, 6) for v in (0.02, 0.20, 0.19)]
-    # choice scores may be negative: a kept output below zero still beats the ones that were ruled out
+    # output 5 chooses at -0.62: below zero, and still ahead of everything in the group that was dropped
     corr2 = torch.tensor([-0.5, -0.9, 0.0, -3.0, 0.5, -0.9], dtype=torch.float64)
     assert [i for i, _ in plain.choose(logits, corr2, {"groups": {"count": 3, "keep": 2}, "top": 4})] == [4, 2, 5, 3]
 

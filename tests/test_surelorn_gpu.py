@@ -41,7 +41,7 @@ def test_embedding_with_sinusoid(dtype, width):
     assert torch.allclose(x.cpu().double(), want, atol=2e-6) and torch.equal(h.cpu(), x.cpu().to(dtype))
 
 
-@pytest.mark.parametrize("D", [96, 320, 4096, 130, 33])
+@pytest.mark.parametrize("D", [96, 352, 4096, 6144, 130, 33])
 @pytest.mark.parametrize("dtype", [BF, F32])
 def test_stream_update_and_final_norm(D, dtype):
     N, P, top = 11, 20, 3
@@ -133,7 +133,7 @@ def _attend(q, lat, pos, scale):
     return torch.softmax(s, -1) @ lat[:pos + 1]
 
 
-SHAPES = [(128, 4), (128, 17), (96, 3), (64, 33), (512, 16), (512, 40), (256, 64), (72, 5), (384, 8), (36, 6), (40, 2), (33, 3), (1024, 2)]
+SHAPES = [(128, 6), (128, 17), (96, 3), (64, 33), (512, 16), (512, 40), (256, 64), (72, 5), (384, 8), (36, 6), (40, 2), (33, 3), (1024, 2)]
 
 
 @pytest.mark.parametrize("rank,heads", SHAPES)
@@ -161,7 +161,7 @@ def test_latent_attention_over_pages(rank, heads, dtype):
         assert float((got - want).abs().max()) < tol * float(want.abs().max())
 
 
-@pytest.mark.parametrize("rank,heads", [(128, 4), (512, 20), (256, 40), (36, 3)])
+@pytest.mark.parametrize("rank,heads", [(128, 6), (512, 20), (256, 40), (36, 3)])
 def test_one_standing_out_key_is_found_anywhere_and_the_next_one_is_not_seen(rank, heads):
     n = 1100
     for dtype in (BF, F32):
@@ -235,7 +235,7 @@ def test_routing(experts, identity, top, groups, keep):
 
 
 @pytest.mark.parametrize("N,D,F,E,identity,top", [(1, 64, 32, 4, 1, 2), (7, 96, 40, 6, 2, 3), (300, 128, 64, 5, 3, 2), (40, 256, 160, 70, 2, 6), (513, 64, 96, 3, 0, 1),
-                                                  (50, 130, 30, 5, 1, 2), (2000, 320, 64, 12, 2, 4)])
+                                                  (50, 130, 30, 5, 1, 2), (2000, 352, 96, 10, 2, 3)])
 @pytest.mark.parametrize("dtype", [BF, F32])
 def test_expert_outputs(N, D, F, E, identity, top, dtype):
     h, gu, dn = rand(N, D, seed=1, dtype=dtype), rand(E, 2 * F, D, seed=2, dtype=dtype, scale=D ** -0.5), rand(E, D, F, seed=3, dtype=dtype, scale=F ** -0.5)
