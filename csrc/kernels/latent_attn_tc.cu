@@ -77,7 +77,7 @@ struct LtSmem {
 };
 
 template <int NP>
-__global__ void __launch_bounds__(LT_THREADS)
+__global__ void __launch_bounds__(LT_THREADS, NP == 64 ? 1 : 2)
 latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const LatentTcDev a) {
   using S = LtSmem<NP>;
   constexpr int CPT = NP / 2, TS = (int)S::T_STRIDE;
@@ -300,29 +300,38 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const Latent
     }
     if (ok) {
       tc_fence_after();
+      // everything that depends on the column alone is worked out once; the stores below are an addition each
+      float inv[CPT];
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) {
+        const int hr = half * CPT + j;
+        const float l = lred[hr] + lred[NP + hr] + lred[2 * NP + hr] + lred[3 * NP + hr];
+        inv[j] = 1.0f / l;
+        if (a.splits > 1 && kin == 0 && hr < nh) {
+          float* ml = a.ml + ((t * c.heads + h0 + hr) * a.splits + split) * 2;
+          ml[0] = stat[hr];
+          ml[1] = l;
+        }
+      }
+      const long long row0 = t * c.heads + h0 + half * CPT;
+      __nv_bfloat16* out = a.out + row0 * R + kin;
+      float* part = a.part + (row0 * a.splits + split) * R + kin;
+      const int step = a.splits * R, mine = nh - half * CPT;         // columns of this half that are heads
       for (int m = 0; m < ns; ++m) {
         uint32_t o[CPT], lo[CPT];
         __syncwarp();
         lt_ld<CPT>(t_s + NP * (1 + 2 * m), o);
         lt_ld<CPT>(t_s + NP * (2 + 2 * m), lo);
         tmem_ld_wait();
-        const int r = m * 128 + kin;
+        if (m * 128 + kin >= R) continue;
+        if (a.splits == 1) {
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) {
-          const int hr = half * CPT + j;
-          if (hr >= nh || r >= R) continue;
-          const float ov = __uint_as_float(o[j]) + __uint_as_float(lo[j]);
-          const float l = lred[hr] + lred[NP + hr] + lred[2 * NP + hr] + lred[3 * NP + hr];
-          const long long row = t * c.heads + h0 + hr;
-          if (a.splits == 1) {
-            a.out[row * R + r] = __float2bfloat16(ov / l);
-          } else {
-            a.part[(row * a.splits + split) * R + r] = ov;
-            if (r == 0) {
-              a.ml[(row * a.splits + split) * 2] = stat[hr];
-              a.ml[(row * a.splits + split) * 2 + 1] = l;
-            }
-          }
+          for (int j = 0; j < CPT; ++j)
+            if (j < mine) out[m * 128 + j * R] = __float2bfloat16((__uint_as_float(o[j]) + __uint_as_float(lo[j])) * inv[j]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < CPT; ++j)
+            if (j < mine) part[m * 128 + j * step] = __uint_as_float(o[j]) + __uint_as_float(lo[j]);
         }
       }
     }

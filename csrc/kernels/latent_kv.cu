@@ -142,7 +142,11 @@ latent_attention_kernel(const LatentDev c, const T* __restrict__ q, T* __restric
 __global__ void latent_merge_kernel(const float* __restrict__ part, const float* __restrict__ ml, __nv_bfloat16* __restrict__ out, int splits, int R) {
   __shared__ float weight[32];
   const long long row = blockIdx.x;
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & 31, r = blockIdx.y * blockDim.x + threadIdx.x;
+  const float* p = part + row * splits * R + r;
+  float e[16];                                       // the first ranges' sums travel while the weights are worked out
+#pragma unroll
+  for (int s = 0; s < 16; ++s) e[s] = (s < splits && r < R) ? p[(long long)s * R] : 0.0f;
   if (threadIdx.x < 32) {
     const float2 v = lane < splits ? reinterpret_cast<const float2*>(ml)[row * splits + lane] : make_float2(-INFINITY, 0.0f);
     const float m = warp_max(v.x);
@@ -150,14 +154,17 @@ __global__ void latent_merge_kernel(const float* __restrict__ part, const float*
     weight[lane] = f / warp_sum(v.y * f);
   }
   __syncthreads();
-  const float* p = part + row * splits * R;
-  const int r = blockIdx.y * blockDim.x + threadIdx.x;
   if (r >= R) return;
+  // a range without keys has weight 0 and wrote no sums: whatever its memory holds is not used
   float v = 0.0f;
-#pragma unroll 16
-  for (int s = 0; s < splits; ++s) {
-    const float e = p[(long long)s * R + r], w = weight[s];
-    v += w > 0.0f ? w * e : 0.0f;                    // a range without keys wrote no sums: its memory is not looked at
+#pragma unroll
+  for (int s = 0; s < 16; ++s) {
+    const float w = weight[s];
+    v += w > 0.0f ? w * e[s] : 0.0f;
+  }
+  for (int s = 16; s < splits; ++s) {
+    const float w = weight[s];
+    v += w > 0.0f ? w * p[(long long)s * R] : 0.0f;
   }
   out[row * R + r] = __float2bfloat16(v);
 }
