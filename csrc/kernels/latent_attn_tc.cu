@@ -41,10 +41,9 @@ __device__ __forceinline__ void lt_ld(uint32_t taddr, uint32_t (&r)[N]) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
                  : "r"(taddr)
                  : "memory");
-  } else if constexpr (N == 16) {
-    tmem_ld16(taddr, r);
   } else {
-    tmem_ld32(taddr, r);
+    static_assert(N == 16, "8 or 16 columns");
+    tmem_ld16(taddr, r);
   }
 }
 template <int N>
@@ -53,10 +52,9 @@ __device__ __forceinline__ void lt_st(uint32_t taddr, const uint32_t (&r)[N]) {
     asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};"
                  ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7])
                  : "memory");
-  } else if constexpr (N == 16) {
-    tmem_st16(taddr, r);
   } else {
-    tmem_st32(taddr, r);
+    static_assert(N == 16, "8 or 16 columns");
+    tmem_st16(taddr, r);
   }
 }
 // meeting point of the eight softmax warps
@@ -77,7 +75,7 @@ struct LtSmem {
 };
 
 template <int NP>
-__global__ void __launch_bounds__(LT_THREADS, NP == 64 ? 1 : 2)
+__global__ void __launch_bounds__(LT_THREADS, 2)
 latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_pages, const LatentTcDev a) {
   using S = LtSmem<NP>;
   constexpr int CPT = NP / 2, TS = (int)S::T_STRIDE;
@@ -381,9 +379,10 @@ int launch_latent_tc(const LatentDev& d, const __nv_bfloat16* q, __nv_bfloat16* 
   uint32_t box[3] = {64, 64, 1};
   int rc = encode_tmap(&tm, d.pages, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, strides, box, Swz::B128);
   if (rc) return rc;
-  if (d.heads <= 16) rc = launch_np<16>(tm, a, rows, st);
-  else if (d.heads <= 32 || a.ns > 2) rc = launch_np<32>(tm, a, rows, st);
-  else rc = launch_np<64>(tm, a, rows, st);
+  // 16 heads per CTA while that leaves every CTA an SM (a CTA's time grows with its heads), else 32: more heads share
+  // one pass over the latents, and the per-thread state of a wider tile no longer fits in registers
+  if (d.heads <= 16 || (long long)rows * ((d.heads + 15) / 16) * splits <= sm_count(dev)) rc = launch_np<16>(tm, a, rows, st);
+  else rc = launch_np<32>(tm, a, rows, st);
   if (rc) return rc;
   if (splits > 1) CGK_CUDA_CHECK(launch_latent_merge(a.part, a.ml, out, rows * d.heads, splits, d.R, st));
   return 0;
