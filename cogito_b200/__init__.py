@@ -19,6 +19,7 @@ _NAMES = {
     # models
     "GPT2": "models.gpt2", "GPT2Config": "models.gpt2", "Llama": "models.llama", "LlamaConfig": "models.llama",
     "Surelorn": "models.surelorn", "SurelornConfig": "models.surelorn", "load_folder": "models.registry",
+    "Nufalorn": "models.nufalorn", "NufalornConfig": "models.nufalorn", "save_folder": "models.registry", "HybridCache": "serve.hybrid_cache",
     "MLPClassifier": "models.mlp", "XorNet": "models.mlp", "ConvClassifier": "models.cnn",
     # training
     "Trainer": "train", "FusedAdam": "optim.fused", "FusedSGD": "optim.fused", "GradScaler": "optim.fused",

@@ -34,7 +34,7 @@ TRAIN = {
                                                                        device=dev, dtype=dt)),
 }
 # architecture -> class with ``from_folder(path, device, dtype)``; these run in serve.stack.StackEngine
-SERVE = {"Surelorn": "models.surelorn:Surelorn"}
+SERVE = {"Surelorn": "models.surelorn:Surelorn", "Nufalorn": "models.nufalorn:Nufalorn"}
 
 
 def train_config(family: str, section: dict):
@@ -57,3 +57,12 @@ def load_folder(path: str, device="cuda", dtype=None):
         raise ValueError(f"{path}: no model class for architecture {name!r} (known: {', '.join(SERVE)})")
     kw = {} if dtype is None else {"dtype": dtype}
     return _cls(SERVE[name]).from_folder(path, device, **kw)
+
+
+def save_folder(path: str, cfg, tensors) -> None:
+    """Writes config.json (``cfg.to_dict()``) and model.safetensors, what ``load_folder`` reads."""
+    from ..io.safetensors import save_safetensors
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg.to_dict(), f, indent=1)
+    save_safetensors(os.path.join(path, "model.safetensors"), tensors)

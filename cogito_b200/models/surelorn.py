@@ -21,6 +21,8 @@ from ..nn.latent_attention import LatentAttention, LatentSpec, _frozen
 from ..nn.moe import DenseSpec, GatedMLP, MixtureOfExperts, MoESpec
 from ..ops import stream as S
 from ..ops.linear import linear
+from ..serve.kv_cache import PagedLatentCache
+from .registry import save_folder  # noqa: F401
 
 POSITION_BASE = 10000.0
 
@@ -189,8 +191,8 @@ class Surelorn(nn.Module):
         self.runs = [self.sets[str(cfg.home(i))] for i in range(len(cfg.layers))]
 
     # ------------------------------------------------------------ what an engine asks of a model
-    def cache_ranks(self) -> list[int]:
-        return [l.attn.cache_rank for l in self.runs]
+    def new_cache(self, batch: int, max_seq_len: int, page_size: int, n_pages: int | None = None) -> PagedLatentCache:
+        return PagedLatentCache([l.attn.cache_rank for l in self.runs], batch, max_seq_len, page_size, self.device, self.dtype, n_pages)
 
     def vocab(self) -> int:
         return self.cfg.vocab_size
@@ -224,10 +226,3 @@ class Surelorn(nn.Module):
             cfg = SurelornConfig.from_dict(json.load(f))
         return cls(cfg, load_safetensors(os.path.join(path, "model.safetensors")), device, dtype)
 
-
-def save_folder(path: str, cfg: SurelornConfig, tensors: dict[str, torch.Tensor]) -> None:
-    from ..io.safetensors import save_safetensors
-    os.makedirs(path, exist_ok=True)
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg.to_dict(), f, indent=1)
-    save_safetensors(os.path.join(path, "model.safetensors"), tensors)

@@ -1,4 +1,4 @@
-"""Gated feed-forward layers of inference models: dense (silu(gate) * up) and mixture of experts with a softmax
+"""Gated feed-forward layers of inference models: dense (act(gate) * up, act silu or relu) and mixture of experts with a softmax
 router, an additive correction that steers the choice only, group-limited selection, identity outputs and a shared
 expert that every token takes."""
 from __future__ import annotations
@@ -34,16 +34,21 @@ class MoESpec:
 
 
 class GatedMLP(nn.Module):
-    """W_down (silu(W_gate h) * (W_up h)); the gate and up products are one product."""
+    """W_down (act(W_gate h) * (W_up h)); the gate and up products are one product."""
 
-    def __init__(self, tensors, device, dtype):
+    def __init__(self, tensors, device, dtype, act: str = "silu"):
         super().__init__()
         t = {k: v.to(device) for k, v in tensors.items()}
+        self.act = act
         self.w_gate_up = _frozen(torch.cat([t["gate"], t["up"]], 0).to(dtype).contiguous())
         self.w_down = _frozen(t["down"].to(dtype).contiguous())
 
+    def inner(self, h, out=None):
+        """act(W_gate h) * (W_up h), what W_down is applied to."""
+        return gated_linear(h, self.w_gate_up, self.act, out)
+
     def forward(self, h):
-        return linear(gated_linear(h, self.w_gate_up), self.w_down)
+        return linear(self.inner(h), self.w_down)
 
     def branch(self, h):
         """What the stream update adds: (dense result, no expert rows)."""

@@ -22,7 +22,7 @@ if not _DEBUG and not _LIB_PATH.exists() and (_LIB_DIR / "libcogito_kernels_serv
 _lib = None
 # source files that carry index checks in the debug build (one recorded violation each)
 _BOUNDS_FILES = ("gemm_tcgen05", "softmax_ce", "serving", "elementwise", "flash_fwd", "flash_bwd", "residual_stream", "latent_kv",
-                 "latent_attn_tc", "moe")
+                 "latent_attn_tc", "moe", "kv_rows", "linear_state")
 
 
 class KernelError(RuntimeError):
@@ -118,6 +118,14 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_moe_gather": [vp, vp, i, i, i, vp, vp, vp, i, i, vp],
         "cgk_gemm_grouped_bf16": [POINTER(GemmArgs), vp, vp, vp],
         "cgk_swiglu_tiles": [vp, vp, vp, i, i, vp],
+        "cgk_rotary_angles": [vp, vp, vp, i, i, vp],
+        "cgk_kv_rotate_append": [vp, vp, i, vp],
+        "cgk_kv_gather": [vp, i, i, i, i, vp, vp, vp],
+        "cgk_kv_rows_attention": [vp, vp, ll, i, vp, ll, vp, i, i, f, i, i, i, vp, vp],
+        "cgk_linear_state": [vp, i, vp],
+        "cgk_stream_norms": [vp, vp],
+        "cgk_softcap": [vp, ll, f, vp],
+        "cgk_gated_rows": [i, vp, vp, ll, ll, i, i, vp],
         "cgk_expert_rows": [i, vp, vp, i, i, i, vp, vp, vp, vp, i, i, vp],
     }
     for name, argtypes in sigs.items():
@@ -133,6 +141,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_int4_wa_tiles_bytes": [i, i],
         "cgk_int4_gemm_counters": [i, i],
         "cgk_latent_attention_scratch_floats": [i, i, i, i],
+        "cgk_kv_rows_scratch_floats": [i, i, i, i],
     }.items():
         fn = getattr(L, name, None)
         if fn is None:                              # a library built from part of the sources

@@ -34,6 +34,7 @@ class FlashArgs(Structure):
         ("dk_bs", c_int64), ("dk_ts", c_int64), ("dk_hs", c_int64),
         ("dv_bs", c_int64), ("dv_ts", c_int64), ("dv_hs", c_int64),
         ("delta", c_void_p), ("dq_accum", c_void_p),
+        ("block", c_int32), ("sink", c_int32), ("turn", c_void_p), ("o_cols", c_int32),
     ]
 
 
@@ -58,7 +59,7 @@ def alibi_slopes(num_heads: int, device=None) -> torch.Tensor:
     return torch.pow(2.0, -8.0 * h / num_heads)
 
 
-def attention_reference(q, k, v, *, causal=False, window=-1, scale=None, alibi=None):
+def attention_reference(q, k, v, *, causal=False, window=-1, scale=None, alibi=None, block=0, sink=False):
     """Naive softmax(QK^T)V in fp32 with the same masking rules; returns (o, lse)."""
     B, Tq, Hq, D = q.shape
     Tk, Hk = k.shape[1], k.shape[2]
@@ -77,8 +78,12 @@ def attention_reference(q, k, v, *, causal=False, window=-1, scale=None, alibi=N
         vis &= ki <= qi
     if window is not None and window >= 0:
         vis &= (ki - qi).abs() <= window
+    if block:
+        vis &= torch.div(ki, block, rounding_mode="floor") == torch.div(qi, block, rounding_mode="floor")
     s = s.masked_fill(~vis, float("-inf"))
     lse = torch.logsumexp(s, dim=-1)
+    if sink:
+        lse = torch.logaddexp(lse, torch.zeros_like(lse))
     p = torch.exp(s - lse.masked_fill(torch.isinf(lse), 0.0).unsqueeze(-1))
     p = torch.nan_to_num(p, nan=0.0)
     o = torch.matmul(p, vf).permute(0, 2, 1, 3)
@@ -106,13 +111,24 @@ def _fill_common(a: FlashArgs, q, k, v, o, lse, scale, causal, window, alibi):
     a.alibi_slopes = alibi.data_ptr() if alibi is not None else None
 
 
-def flash_forward(q, k, v, *, causal=False, window=-1, scale=None, alibi=None, out=None):
+def turn_back(o, turn):
+    """o [.., heads, n], turn [.., n / 2, 2] (cos, sin): pairs (2i, 2i + 1) turned by minus the angle."""
+    u, v = o[..., 0::2], o[..., 1::2]
+    c, s = turn[..., 0].unsqueeze(-2), turn[..., 1].unsqueeze(-2)
+    return torch.stack([u * c + v * s, v * c - u * s], -1).flatten(-2)
+
+
+def flash_forward(q, k, v, *, causal=False, window=-1, scale=None, alibi=None, out=None, block=0, sink=False, turn=None):
     """Returns (o [B,Tq,Hq,D] bf16, lse [B,Hq,Tq] fp32).  q/k/v may be strided views; ``out`` (same shape as q,
-    may be a strided view) receives o."""
+    may be a strided view, may keep only the first elements of every head) receives o.
+    block > 0: with ``causal``, a query sees the keys of its own block of that many (counted from key 0).  sink: one is
+    added to the softmax denominator.  turn: fp32 [B, Tq, n / 2, 2] (cos, sin), the n elements of ``out`` are turned back."""
     B, Tq, Hq, D = q.shape
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     if not q.is_cuda:
-        o, lse = attention_reference(q, k, v, causal=causal, window=window, scale=scale, alibi=alibi)
+        o, lse = attention_reference(q, k, v, causal=causal, window=window, scale=scale, alibi=alibi, block=block, sink=sink)
+        o = o if out is None else o[..., :out.shape[-1]]
+        o = o if turn is None else turn_back(o, turn)
         if out is not None:
             return out.copy_(o), lse
         return o.to(q.dtype), lse
@@ -122,6 +138,9 @@ def flash_forward(q, k, v, *, causal=False, window=-1, scale=None, alibi=None, o
     lse = torch.empty(B, Hq, Tq, device=q.device, dtype=torch.float32)
     a = FlashArgs()
     _fill_common(a, q, k, v, o, lse, scale, causal, window, alibi)
+    a.block, a.sink = int(block), int(bool(sink))
+    if turn is not None or o.shape[-1] != D:
+        a.turn, a.o_cols = _lib.ptr(turn), o.shape[-1]
     _lib.check(_fns().cgk_flash_forward(ctypes.byref(a), _lib.stream_ptr()), "cgk_flash_forward")
     _lib.count_launch()
     return o, lse

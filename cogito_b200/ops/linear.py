@@ -39,9 +39,12 @@ def linear(a, w, *, w_mn: bool = False, out=None, out_dtype=torch.bfloat16):
     return _skinny(a, w, out, 2 if w_mn else 0, N)
 
 
-def gated_linear(a, w_gate_up):
-    """silu(a W_gate^T) * (a W_up^T); w_gate_up [2F, K]: gate rows, then up rows."""
+def gated_linear(a, w_gate_up, act: str = "silu", out=None):
+    """act(a W_gate^T) * (a W_up^T); w_gate_up [2F, K]: gate rows, then up rows; act silu or relu; out may be a view
+    with longer rows."""
     if not _few(a, w_gate_up, False):
-        return M.swiglu(gemm(a, w_gate_up))
+        return M.gated(gemm(a, w_gate_up), act, out)
     F = w_gate_up.shape[0] // 2
-    return _skinny(a, w_gate_up, torch.empty(a.shape[0], F, dtype=a.dtype, device=a.device), 1, F)
+    if out is None:
+        out = torch.empty(a.shape[0], F, dtype=a.dtype, device=a.device)
+    return _skinny(a, w_gate_up, out, 3 if act == "relu" else 1, F)

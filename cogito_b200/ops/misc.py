@@ -122,6 +122,26 @@ def swiglu(x):
     return _SwiGLU.apply(x)
 
 
+GATED = {"silu": 0, "relu": 1}
+
+
+def gated(x, act: str = "silu", out=None):
+    """act(x[..., :F]) * x[..., F:] of rows [rows, 2F] (inference); out may be a view with longer rows."""
+    F = x.shape[-1] // 2
+    if not x.is_cuda:
+        g, u = x.float()[..., :F], x.float()[..., F:]
+        y = ((torch.relu(g) if act == "relu" else torch.nn.functional.silu(g)) * u).to(x.dtype)
+        return y if out is None else out.copy_(y)
+    if out is None:
+        out = torch.empty(x.shape[0], F, dtype=x.dtype, device=x.device)
+    if x.dim() != 2 or not x.is_contiguous() or out.stride(-1) != 1:
+        raise ValueError("gated: contiguous rows expected")
+    _lib.check(_lib.lib().cgk_gated_rows(_dt(x), x.data_ptr(), out.data_ptr(), out.stride(0), x.shape[0], F, GATED[act], _lib.stream_ptr()),
+               "cgk_gated_rows")
+    _lib.count_launch()
+    return out
+
+
 # ---------------------------------------------------------------------------
 class _Dropout(torch.autograd.Function):
     @staticmethod

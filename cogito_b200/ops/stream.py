@@ -1,8 +1,9 @@
-"""Operations of decoders with an fp32 residual stream and RMS norms on the OUTPUT of each sublayer.
+"""Operations of decoders with an fp32 residual stream.
 
-``embed_sinusoid`` starts the stream, ``stream_update`` adds a normalised sublayer result (and hands out the
-stream as the next sublayer's operand in the same kernel), ``rms_rows`` is the norm in front of the
-vocabulary projection.  CUDA: csrc/kernels/residual_stream.cu; CPU tensors take an fp32 restatement.
+RMS norms on the OUTPUT of each sublayer: ``embed_sinusoid`` starts the stream, ``stream_update`` adds a normalised
+sublayer result (and hands out the stream as the next sublayer's operand in the same kernel).  RMS norms on the INPUT:
+``stream_norms`` starts the stream or adds a result and hands out up to two normalised copies.  ``rms_rows`` is the norm
+in front of the vocabulary projection, ``softcap`` limits the logits.  CUDA: csrc/kernels/residual_stream.cu; CPU tensors take an fp32 restatement.
 """
 from __future__ import annotations
 
@@ -20,6 +21,14 @@ class StreamUpdateArgs(Structure):
     _fields_ = [("y", c_void_p), ("ldy", c_int64), ("pairs", c_void_p), ("ldp", c_int64), ("row_of", c_void_p), ("weight", c_void_p),
                 ("w", c_void_p), ("x", c_void_p), ("h", c_void_p), ("rows", c_int32), ("D", c_int32), ("top", c_int32),
                 ("pair_rows", c_int32), ("y_fp32", c_int32), ("pairs_fp32", c_int32), ("h_fp32", c_int32), ("eps", c_float)]
+
+
+class StreamNormsArgs(Structure):
+    """Mirror of ``cgk_stream_norms_args`` (include/cogito_kernels.h)."""
+
+    _fields_ = [("ids", c_void_p), ("table", c_void_p), ("y", c_void_p), ("ldy", c_int64), ("w1", c_void_p), ("w2", c_void_p), ("x", c_void_p),
+                ("h1", c_void_p), ("h2", c_void_p), ("rows", c_int32), ("D", c_int32), ("vocab", c_int32), ("table_fp32", c_int32),
+                ("y_fp32", c_int32), ("h_fp32", c_int32), ("mult", c_float), ("eps", c_float)]
 
 
 def sinusoid_frequencies(width: int, base: float = 10000.0, device=None) -> torch.Tensor:
@@ -72,6 +81,41 @@ def stream_update(x, y, w, eps: float, dtype, pairs=None, row_of=None, weight=No
     _lib.check(_lib.lib().cgk_stream_update(ctypes.byref(a), _lib.stream_ptr()), "cgk_stream_update")
     _lib.count_launch()
     return h
+
+
+def stream_norms(x, eps: float, dtype, w1=None, w2=None, y=None, mult: float = 1.0, ids=None, table=None):
+    """x [N, D] fp32, in place: x = table[ids], or x += mult * y, or unchanged.  Returns (h1, h2): the RMS-normed new
+    stream times w1 and times w2 in ``dtype`` (None where the weight is None)."""
+    if not x.is_cuda:
+        if ids is not None:
+            x.copy_(table[ids].float())
+        elif y is not None:
+            x += mult * y.float()
+        n = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)
+        return tuple(None if w is None else (n * w).to(dtype) for w in (w1, w2))
+    N, D = x.shape
+    h = [None if w is None else torch.empty(N, D, dtype=dtype, device=x.device) for w in (w1, w2)]
+    a = StreamNormsArgs()
+    if ids is not None:
+        a.ids, a.table, a.vocab, a.table_fp32 = ids.data_ptr(), table.data_ptr(), table.shape[0], int(table.dtype == torch.float32)
+    if y is not None:
+        a.y, a.ldy, a.y_fp32 = y.data_ptr(), y.stride(0), int(y.dtype == torch.float32)
+    a.w1, a.w2, a.x, a.h1, a.h2 = _lib.ptr(w1), _lib.ptr(w2), x.data_ptr(), _lib.ptr(h[0]), _lib.ptr(h[1])
+    a.rows, a.D, a.h_fp32, a.mult, a.eps = N, D, int(dtype == torch.float32), float(mult), float(eps)
+    _lib.check(_lib.lib().cgk_stream_norms(ctypes.byref(a), _lib.stream_ptr()), "cgk_stream_norms")
+    _lib.count_launch()
+    return tuple(h)
+
+
+def softcap(x, cap: float):
+    """cap * tanh(x / cap), in place (fp32)."""
+    if not x.is_cuda:
+        return x.copy_(cap * torch.tanh(x / cap))
+    if not x.is_contiguous():
+        raise ValueError("softcap: contiguous logits expected")
+    _lib.check(_lib.lib().cgk_softcap(x.data_ptr(), x.numel(), float(cap), _lib.stream_ptr()), "cgk_softcap")
+    _lib.count_launch()
+    return x
 
 
 def rms_rows(x, w, eps: float, dtype, rows=None):

@@ -243,6 +243,10 @@ class SpeculativeDecoder:
                  top_k: int = 50, top_p: float = 0.9, seed: int = 0, use_graph: bool | None = None):
         if draft.cfg.vocab_size != target.cfg.vocab_size or draft.batch != target.batch:
             raise ValueError("draft and target must share vocabulary and batch size")
+        for e in (draft, target):
+            back = getattr(e, "rollback", None)
+            if back is not None and back < gamma + 1:
+                raise ValueError(f"an engine that can take back {back} tokens cannot verify {gamma} drafts at a time")
         self.draft, self.target, self.gamma = draft, target, gamma
         self.temperature, self.top_k, self.top_p, self.seed = temperature, top_k, top_p, seed
         self.stats = SpecStats()

@@ -2,8 +2,8 @@
 
 A step takes the next tokens of any set of sequences - prompts, portions of prompts, single decoded tokens - runs
 them as one flat batch against the paged cache and returns the logits asked for.  The model supplies
-``stream(batch, cache)``, ``logits(x, rows)``, ``cache_ranks()`` and ``vocab()``; cache, slots, pages, batch layout and
-decode graphs live here.
+``stream(batch, cache)``, ``logits(x, rows)``, ``new_cache(...)`` and ``vocab()``; slots, pages, batch layout and decode
+graphs live here.
 
 Also usable where a fixed batch advances together (``forward(tokens, commit)``, the interface of
 ``LlamaInt4Engine``): the speculative decoder runs on it unchanged.
@@ -17,7 +17,6 @@ from types import SimpleNamespace
 import torch
 
 from ..ops import _lib
-from .kv_cache import PagedLatentCache
 
 
 @dataclass(frozen=True)
@@ -34,13 +33,17 @@ class Segment:
 @dataclass
 class TokenBatch:
     """The flat token batch of a step: ids int64, pos and slot int32, all [N] on the device.  ``prompts`` cover rows
-    [0, single_from); the rows after that are handled token by token.  max_len bounds every sequence's length."""
+    [0, single_from); the rows after that are handled token by token.  max_len bounds every sequence's length.
+    runs [n, 2] int32 on the device: first row and length of every stretch of consecutive tokens of one sequence, the
+    prompts' first (None: every row is one).  memo: what layers of one step share."""
     ids: torch.Tensor
     pos: torch.Tensor
     slot: torch.Tensor
     prompts: list[Segment] = field(default_factory=list)
     single_from: int = 0
     max_len: int = 1
+    runs: torch.Tensor | None = None
+    memo: dict = field(default_factory=dict)
 
 
 class StackEngine:
@@ -57,7 +60,9 @@ class StackEngine:
         if self.pooled:
             # every live sequence may leave its last page partly empty; one more slot takes the padding rows of graphs
             kw["n_pages"] = (pool_tokens + page_size - 1) // page_size + batch + 1
-        self.cache = PagedLatentCache(model.cache_ranks(), batch + (1 if self.pooled else 0), max_seq_len, page_size, self.device, self.dtype, **kw)
+        self.cache = model.new_cache(batch + (1 if self.pooled else 0), max_seq_len, page_size, **kw)
+        # tokens that a caller of ``forward`` may take back after committing them (None: any number)
+        self.rollback = self.cache.history - 1 if hasattr(self.cache, "history") else None
         env = os.environ.get("COGITO_SERVE_GRAPH", "1") != "0"
         self.use_graph = (self.device.type == "cuda" and env and self.pooled) if use_graph is None else use_graph
         self._graphs: dict[tuple[int, int], dict] = {}
@@ -108,7 +113,7 @@ class StackEngine:
         else:
             # prompt portions first; the caller's order of the wanted logits is kept by the row list
             order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]) < self.PROMPT_MIN)
-            ids, pos, slot, segs, single = [], [], [], [], None
+            ids, pos, slot, segs, runs, single = [], [], [], [], [], None
             first = {}
             for i in order:
                 s, toks, _ = entries[i]
@@ -118,13 +123,15 @@ class StackEngine:
                     segs.append(Segment(len(ids), 1, n, s, begin))
                 elif single is None:
                     single = len(ids)
+                runs.append((len(ids), n))
                 ids += toks
                 pos += range(begin, begin + n)
                 slot += [s] * n
             host = torch.tensor([ids, pos, slot], dtype=torch.int64)
             dev = host.to(self.device)
             small = dev[1:].to(torch.int32)
-            batch = TokenBatch(dev[0], small[0], small[1], segs, len(ids) if single is None else single, max(pos) + 1)
+            batch = TokenBatch(dev[0], small[0], small[1], segs, len(ids) if single is None else single, max(pos) + 1,
+                               torch.tensor(runs, dtype=torch.int32).to(self.device))
             x = self.model.stream(batch, self.cache, **({} if keep is None else {"keep": keep}))
             rows = [first[i] + w for i, (_, _, want) in enumerate(entries) for w in want]
             out = torch.empty(0, V, device=self.device)
@@ -196,6 +203,9 @@ class StackEngine:
         pos = (self.cache.lengths[:, None] + torch.arange(T, device=dev, dtype=torch.int32)[None]).reshape(-1)
         slot = torch.arange(B, device=dev, dtype=torch.int32).repeat_interleave(T)
         batch = TokenBatch(tokens.reshape(-1).long(), pos, slot, max_len=self.max_seq_len)
+        if T > 1:
+            first = torch.arange(0, B * T, T, device=dev, dtype=torch.int32)
+            batch.runs = torch.stack([first, torch.full_like(first, T)], 1)
         if fresh:
             batch.prompts, batch.single_from = [Segment(0, B, T, 0, 0)], B * T
         logits = self.model.logits(self.model.stream(batch, self.cache)).view(B, T, -1)

@@ -371,20 +371,21 @@ __global__ void dropout_kernel(const T* __restrict__ x, T* out, long long n, flo
 }
 
 // ---- SwiGLU: x = [rows, 2H] as (gate | value); y = silu(gate) * value ----------
-template <typename T>
-__global__ void swiglu_fwd_kernel(const T* __restrict__ x, T* __restrict__ y, long long rows, int H) {
+template <typename T, int ACT>
+__global__ void swiglu_fwd_kernel(const T* __restrict__ x, T* __restrict__ y, long long ldo, long long rows, int H) {
   const long long n = rows * H;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n;
        i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / H;
     const int c = (int)(i - r * H);
     const float g = ldf<T>(x, r * 2 * H + c), v = ldf<T>(x, r * 2 * H + H + c);
-    stf<T>(y, i, silu_f(g) * v);
+    stf<T>(y, r * ldo + c, gated_act<ACT>(g) * v);
   }
 }
+template <int ACT>
 __global__ void __launch_bounds__(256)
-swiglu_fwd_rows_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ y, long long rows, int H) {
-  swiglu_rows_bf16(x, y, rows, H);
+swiglu_fwd_rows_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ y, long long ldo, long long rows, int H) {
+  swiglu_rows_bf16<ACT>(x, y, ldo, rows, H);
 }
 template <typename T>
 __global__ void swiglu_bwd_kernel(const T* __restrict__ x, const T* __restrict__ dy,
@@ -725,15 +726,25 @@ CGK_API int cgk_dropout(int dtype, const void* x, void* out, long long n, float 
   return 0;
 }
 
-CGK_API int cgk_swiglu_forward(int dtype, const void* x, void* y, long long rows, int H, void* stream) {
-  CGK_REQUIRE(x && y && H > 0, "cgk_swiglu_forward: bad argument");
+template <int ACT>
+static int launch_gated(int dtype, const void* x, void* y, long long ldo, long long rows, int H, cudaStream_t st) {
   if (rows == 0) return 0;
-  if (dtype == 0) swiglu_fwd_kernel<float><<<ew_grid(rows * H), 256, 0, ST(stream)>>>((const float*)x, (float*)y, rows, H);
-  else if (H % 8 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0)
-    swiglu_fwd_rows_kernel<<<swiglu_rows_grid(rows, H), swiglu_rows_threads(H), 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
-  else swiglu_fwd_kernel<__nv_bfloat16><<<ew_grid(rows * H), 256, 0, ST(stream)>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, H);
+  typedef __nv_bfloat16 bf;
+  if (dtype == 0) swiglu_fwd_kernel<float, ACT><<<ew_grid(rows * H), 256, 0, st>>>((const float*)x, (float*)y, ldo, rows, H);
+  else if (H % 8 == 0 && ldo % 8 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0)
+    swiglu_fwd_rows_kernel<ACT><<<swiglu_rows_grid(rows, H), swiglu_rows_threads(H), 0, st>>>((const bf*)x, (bf*)y, ldo, rows, H);
+  else swiglu_fwd_kernel<bf, ACT><<<ew_grid(rows * H), 256, 0, st>>>((const bf*)x, (bf*)y, ldo, rows, H);
   CGK_LAUNCH_CHECK();
   return 0;
+}
+CGK_API int cgk_swiglu_forward(int dtype, const void* x, void* y, long long rows, int H, void* stream) {
+  CGK_REQUIRE(x && y && H > 0, "cgk_swiglu_forward: bad argument");
+  return launch_gated<GATED_SILU>(dtype, x, y, H, rows, H, ST(stream));
+}
+CGK_API int cgk_gated_rows(int dtype, const void* gu, void* out, long long ldo, long long rows, int F, int act, void* stream) {
+  CGK_REQUIRE(gu && out && F > 0 && ldo >= F && rows >= 0 && (act == GATED_SILU || act == GATED_RELU), "cgk_gated_rows: bad argument");
+  return act == GATED_RELU ? launch_gated<GATED_RELU>(dtype, gu, out, ldo, rows, F, ST(stream))
+                           : launch_gated<GATED_SILU>(dtype, gu, out, ldo, rows, F, ST(stream));
 }
 CGK_API int cgk_swiglu_backward(int dtype, const void* x, const void* dy, void* dx, long long rows, int H,
                                 void* stream) {

@@ -20,7 +20,8 @@
 // function; every tile then takes the one short row loop (three-input maxima,
 // packed two-wide fp32 multiply-adds and sums), which keeps the hot code small.
 //
-// Supports causal masking (bottom-right aligned when Tq != Tk), a sliding window
+// Supports causal masking (bottom-right aligned when Tq != Tk), blocks of keys that only see themselves, a sink (one
+// more term of 1 in the softmax denominator), results turned back by rotary angles, a sliding window
 // |k - q| <= w, ALiBi slopes, GQA/MQA (kv head = h * Hk / Hq), head_dim 64 / 128.
 // Layout [batch, seq, heads, head_dim] with arbitrary (16-byte aligned) strides,
 // LSE [batch, heads, seq] as in the reference (include/cg_flash_attn.h:54-57,81).
@@ -44,6 +45,10 @@ struct FlashFwdDev {
   __nv_bfloat16* O;
   long long o_bs, o_ts, o_hs;  // element strides of O: batch, token, head
   float* lse;              // [B, Hq, Tq] or null
+  int block;               // > 0: causal inside blocks of this many keys
+  int sink;
+  const float2* turn;      // [B * Tq][o_cols / 2] or null
+  int o_cols, o_vec;       // columns stored; 1: rows take 16-byte stores
   int* status;
 };
 
@@ -127,6 +132,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     int first = q0 + off - p.window;
     lo = first > 0 ? first / C::BN : 0;
   }
+  if (p.block > 0 && q0 + off > 0) lo = (q0 + off) / p.block * p.block / C::BN;
   int hi_t[2];
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
@@ -329,6 +335,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       bool need_mask = (k0 + C::BN > p.Tk);
       if (p.causal) need_mask |= (k0 + C::BN - 1 > tile_q_lo);
       if (p.window >= 0) need_mask |= (k0 < tile_q_hi - p.window) || (!p.causal && k0 + C::BN - 1 > tile_q_lo + p.window);
+      if (p.block > 0) need_mask |= k0 < tile_q_hi / p.block * p.block;
       // Interior tiles (no mask, no bias) use the raw products; the others are first rewritten in
       // TMEM as final log2-domain scores (-inf where masked), after which the multiplier is 1.
       const bool fast = !need_mask && !p.alibi && p.scale_log2 > 0.0f;
@@ -338,6 +345,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         int klo = 0, khi = p.Tk - 1;
         if (p.causal) khi = min(khi, qk);
         if (p.window >= 0) { klo = max(klo, qk - p.window); khi = min(khi, qk + p.window); }
+        if (p.block > 0 && qk > 0) klo = max(klo, qk / p.block * p.block);
         const unsigned span = khi >= klo ? (unsigned)(khi - klo) : 0u;
         const float bias0 = p.alibi ? slope * (float)(k0 - qk) : 0.0f;
         flash_mask_scores(s_tmem, p.scale_log2, slope, bias0, k0 - klo, span, khi < klo);
@@ -435,9 +443,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       if (!mbar_wait(o_done(t), (it - 1) & 1u, dead, p.status, 1320 + t)) ok = false;
       tc_fence_after();
     }
+    if (p.sink) l += exp2f(-m);
     const float inv_l = (l > 0.0f) ? 1.0f / l : 0.0f;
     const bool row_ok = qpos < p.Tq;
     __nv_bfloat16* orow = p.O + (long long)b * p.o_bs + (long long)qpos * p.o_ts + (long long)h * p.o_hs;
+    const float2* turn = p.turn && row_ok ? p.turn + ((long long)b * p.Tq + qpos) * (p.o_cols >> 1) : nullptr;
 #pragma unroll 1
     for (int c = 0; c < D / 32; ++c) {
       uint32_t r[32];
@@ -450,14 +460,30 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         for (int i = 0; i < 32; ++i) r[i] = 0u;
       }
       if (row_ok) {
+        if (turn) {
 #pragma unroll
-        for (int q4 = 0; q4 < 4; ++q4) {
-          uint4 v;
-          v.x = pack_bf16x2(__uint_as_float(r[8 * q4]) * inv_l, __uint_as_float(r[8 * q4 + 1]) * inv_l);
-          v.y = pack_bf16x2(__uint_as_float(r[8 * q4 + 2]) * inv_l, __uint_as_float(r[8 * q4 + 3]) * inv_l);
-          v.z = pack_bf16x2(__uint_as_float(r[8 * q4 + 4]) * inv_l, __uint_as_float(r[8 * q4 + 5]) * inv_l);
-          v.w = pack_bf16x2(__uint_as_float(r[8 * q4 + 6]) * inv_l, __uint_as_float(r[8 * q4 + 7]) * inv_l);
-          *reinterpret_cast<uint4*>(orow + c * 32 + q4 * 8) = v;
+          for (int i = 0; i < 16; ++i)
+            if (c * 16 + i < (p.o_cols >> 1)) {
+              const float2 cs = turn[c * 16 + i];
+              const float u = __uint_as_float(r[2 * i]), w = __uint_as_float(r[2 * i + 1]);
+              r[2 * i] = __float_as_uint(u * cs.x + w * cs.y);
+              r[2 * i + 1] = __float_as_uint(w * cs.x - u * cs.y);
+            }
+        }
+        if (p.o_vec) {
+#pragma unroll
+          for (int q4 = 0; q4 < 4; ++q4) {
+            uint4 v;
+            v.x = pack_bf16x2(__uint_as_float(r[8 * q4]) * inv_l, __uint_as_float(r[8 * q4 + 1]) * inv_l);
+            v.y = pack_bf16x2(__uint_as_float(r[8 * q4 + 2]) * inv_l, __uint_as_float(r[8 * q4 + 3]) * inv_l);
+            v.z = pack_bf16x2(__uint_as_float(r[8 * q4 + 4]) * inv_l, __uint_as_float(r[8 * q4 + 5]) * inv_l);
+            v.w = pack_bf16x2(__uint_as_float(r[8 * q4 + 6]) * inv_l, __uint_as_float(r[8 * q4 + 7]) * inv_l);
+            if (c * 32 + q4 * 8 < p.o_cols) *reinterpret_cast<uint4*>(orow + c * 32 + q4 * 8) = v;
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < p.o_cols) orow[c * 32 + i] = __float2bfloat16(__uint_as_float(r[i]) * inv_l);
         }
       }
     }
@@ -513,8 +539,10 @@ CGK_API int cgk_flash_forward(const cgk_flash_args* pa, void* stream) {
   CGK_REQUIRE(a.q && a.k && a.v && a.o, "cgk_flash_forward: null tensor");
   CGK_REQUIRE(a.D == 64 || a.D == 128, "cgk_flash_forward: head_dim %d not supported (64 or 128)", a.D);
   CGK_REQUIRE(a.Hq % a.Hk == 0, "cgk_flash_forward: Hq must be a multiple of Hk");
-  CGK_REQUIRE(a.o_hs % 8 == 0 && a.o_ts % 8 == 0 && a.o_bs % 8 == 0 && ((uintptr_t)a.o & 15) == 0,
-              "cgk_flash_forward: output strides must be multiples of 8 elements");
+  const bool o_vec = a.o_hs % 8 == 0 && a.o_ts % 8 == 0 && a.o_bs % 8 == 0 && ((uintptr_t)a.o & 15) == 0 && a.o_cols % 8 == 0;
+  CGK_REQUIRE(o_vec || a.o_cols > 0, "cgk_flash_forward: output strides must be multiples of 8 elements");
+  CGK_REQUIRE(a.block >= 0 && a.o_cols >= 0 && a.o_cols <= a.D && (a.block == 0 || (a.causal && a.Tk >= a.Tq)) && (!a.turn || (a.o_cols > 0 && a.o_cols % 2 == 0)),
+              "cgk_flash_forward: bad block, turn or o_cols");
   if (a.B == 0 || a.Tq == 0 || a.Hq == 0) return 0;
   int dev = 0;
   CGK_CUDA_CHECK(cudaGetDevice(&dev));
@@ -525,6 +553,11 @@ CGK_API int cgk_flash_forward(const cgk_flash_args* pa, void* stream) {
   p.alibi = a.alibi_slopes;
   p.O = (__nv_bfloat16*)a.o; p.o_bs = a.o_bs; p.o_ts = a.o_ts; p.o_hs = a.o_hs;
   p.lse = a.lse;
+  p.block = a.block;
+  p.sink = a.sink;
+  p.turn = (const float2*)a.turn;
+  p.o_cols = a.o_cols > 0 ? a.o_cols : a.D;
+  p.o_vec = o_vec;
   p.status = device_status(dev);
   if (a.D == 64) return launch_fwd<64>(a, p, (cudaStream_t)stream);
   return launch_fwd<128>(a, p, (cudaStream_t)stream);

@@ -158,7 +158,7 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ h, const int
 // act[row][f] = silu(gu[row][f]) * gu[row][F + f] over the rows in use (*tiles * 128)
 __global__ void __launch_bounds__(256)
 swiglu_tiles_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act, const int* __restrict__ tiles, int F) {
-  swiglu_rows_bf16(gu, act, (long long)*tiles * 128, F);
+  swiglu_rows_bf16(gu, act, F, (long long)*tiles * 128, F);
 }
 
 template <typename T, int V>

@@ -3,7 +3,9 @@
 //   * stream update x += rms(y) * w, where y is a projection's result, or a weighted sum of expert
 //     rows (some of which may stand for the stream itself) plus such a result; the new stream also leaves
 //     as the bf16 (or fp32) operand of the next sublayer,
-//   * RMS norm of selected stream rows (before the vocabulary projection).
+//   * stream start or update x = E[id], x += mult * y, followed by up to two RMS norms of the new stream with weights of their
+//     own (layers whose sublayers read one stream side by side),
+//   * RMS norm of selected stream rows (before the vocabulary projection), soft cap of logits.
 // One CTA per row: a row is read once, kept in shared memory between the statistics and the update.
 #include "../../include/cogito_kernels.h"
 #include "host_common.h"
@@ -188,6 +190,91 @@ stream_update_regs_kernel(const UpdateDev a) {
   }
 }
 
+struct NormsDev {
+  const long long* ids; const void* table; const void* y; long long ldy;
+  const float* w1; const float* w2; float* x; void* h1; void* h2;
+  int D, vocab;
+  float mult, eps;
+};
+
+// V elements per thread and step, the row in registers (ITER steps) or, with ITER 0, in shared memory.
+template <typename TE, typename TY, typename TH, int V, int ITER>
+__global__ void __launch_bounds__(512)
+stream_norms_kernel(const NormsDev a) {
+  extern __shared__ float row_buf[];
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  float* x = a.x + t * a.D;
+  const TE* e = a.ids ? reinterpret_cast<const TE*>(a.table) + CGK_IDX(a.ids[t], a.vocab) * a.D : nullptr;
+  const TY* y = reinterpret_cast<const TY*>(a.y) + t * a.ldy;
+  float xv[ITER > 0 ? ITER : 1][V], ss = 0.0f;
+  auto take = [&](int c, float (&v)[V]) {
+    if constexpr (V == 8) {
+      if (e) { ld8(e + c, v); } else { ld8(x + c, v); }
+    } else {
+      v[0] = e ? ld1(e + c) : x[c];
+    }
+    if (a.y) {
+      float u[V];
+      if constexpr (V == 8) ld8(y + c, u); else u[0] = ld1(y + c);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = fmaf(a.mult, u[j], v[j]);
+    }
+    if (a.y || e) {
+      if constexpr (V == 8) st8(x + c, v); else x[c] = v[0];
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss = fmaf(v[j], v[j], ss);
+  };
+  if constexpr (ITER > 0) {
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < a.D) take(c, xv[i]);
+    }
+  } else {
+    for (int c = threadIdx.x * V; c < a.D; c += blockDim.x * V) {
+      take(c, xv[0]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) row_buf[c + j] = xv[0][j];
+    }
+  }
+  if (!a.h1 && !a.h2) return;
+  ss = block_sum(ss, red);
+  const float r = 1.0f / sqrtf(ss / a.D + a.eps);
+  auto give = [&](int c, const float (&v)[V], const float* w, void* h) {
+    if (!h) return;
+    float o[V];
+    if constexpr (V == 8) {
+      ld8(w + c, o);
+    } else {
+      o[0] = w[c];
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] *= v[j] * r;
+    TH* p = reinterpret_cast<TH*>(h) + t * a.D + c;
+    if constexpr (V == 8) st8(p, o); else st1(p, o[0]);
+  };
+  if constexpr (ITER > 0) {
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < a.D) { give(c, xv[i], a.w1, a.h1); give(c, xv[i], a.w2, a.h2); }
+    }
+  } else {
+    for (int c = threadIdx.x * V; c < a.D; c += blockDim.x * V) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) xv[0][j] = row_buf[c + j];
+      give(c, xv[0], a.w1, a.h1);
+      give(c, xv[0], a.w2, a.h2);
+    }
+  }
+}
+
+__global__ void softcap_kernel(float* __restrict__ x, long long n, float cap, float inv) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) x[i] = cap * tanhf(x[i] * inv);
+}
+
 template <typename TO>
 __global__ void rms_rows_kernel(const float* __restrict__ x, const long long* __restrict__ rows, int n_rows, const float* __restrict__ w,
                                 TO* __restrict__ out, int D, float eps) {
@@ -231,10 +318,56 @@ int launch_update(const UpdateDev& d, int rows, bool vec, cudaStream_t st) {
   return 0;
 }
 
+template <typename TE, typename TY, typename TH>
+int launch_norms(const NormsDev& d, int rows, bool vec, cudaStream_t st) {
+  if (vec && d.D <= 512 * 8 * 4) {
+    const int vecs = d.D / 8, iter = vecs <= 512 ? 1 : (vecs <= 1024 ? 2 : 4), nt = ((vecs + iter - 1) / iter + 31) / 32 * 32;
+    if (iter == 1) stream_norms_kernel<TE, TY, TH, 8, 1><<<rows, nt, 0, st>>>(d);
+    else if (iter == 2) stream_norms_kernel<TE, TY, TH, 8, 2><<<rows, nt, 0, st>>>(d);
+    else stream_norms_kernel<TE, TY, TH, 8, 4><<<rows, nt, 0, st>>>(d);
+  } else {
+    const int smem = d.D * 4;
+    if (smem > 48 * 1024)
+      CGK_CUDA_CHECK(cudaFuncSetAttribute(stream_norms_kernel<TE, TY, TH, 1, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    stream_norms_kernel<TE, TY, TH, 1, 0><<<rows, row_threads(d.D), smem, st>>>(d);
+  }
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
+
 }  // namespace
 }  // namespace cgk
 
 using namespace cgk;
+
+CGK_API int cgk_stream_norms(const cgk_stream_norms_args* pa, void* stream) {
+  CGK_REQUIRE(pa, "cgk_stream_norms: null args");
+  const cgk_stream_norms_args& a = *pa;
+  CGK_REQUIRE(a.x && a.rows >= 0 && a.D > 0 && (!a.ids || (a.table && a.vocab > 0)) && !(a.ids && a.y) && (!a.h1 || a.w1) && (!a.h2 || a.w2),
+              "cgk_stream_norms: bad arguments");
+  CGK_REQUIRE(a.D * 4 <= 200 * 1024, "cgk_stream_norms: rows of %d elements are too long", a.D);
+  if (a.rows == 0) return 0;
+  NormsDev d{(const long long*)a.ids, a.table, a.y, a.ldy, a.w1, a.w2, a.x, a.h1, a.h2, a.D, a.vocab, a.mult, a.eps};
+  auto al = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
+  const bool vec = a.D % 8 == 0 && a.ldy % 8 == 0 && al(a.table) && al(a.y) && al(a.w1) && al(a.w2) && al(a.x) && al(a.h1) && al(a.h2);
+  cudaStream_t st = (cudaStream_t)stream;
+  typedef __nv_bfloat16 bf;
+  if (a.h_fp32) {
+    CGK_REQUIRE((!a.ids || a.table_fp32) && (!a.y || a.y_fp32), "cgk_stream_norms: the fp32 form takes fp32 inputs");
+    return launch_norms<float, float, float>(d, a.rows, vec, st);
+  }
+  CGK_REQUIRE(!a.ids || !a.table_fp32, "cgk_stream_norms: table and norms must have one type");
+  return a.y_fp32 ? launch_norms<bf, float, bf>(d, a.rows, vec, st) : launch_norms<bf, bf, bf>(d, a.rows, vec, st);
+}
+
+CGK_API int cgk_softcap(void* x, long long n, float cap, void* stream) {
+  CGK_REQUIRE((x || n == 0) && n >= 0 && cap > 0.0f, "cgk_softcap: bad arguments");
+  if (n == 0) return 0;
+  const long long blocks = (n + 1023) / 1024;
+  softcap_kernel<<<(unsigned)(blocks < 148 * 16 ? blocks : 148 * 16), 256, 0, (cudaStream_t)stream>>>((float*)x, n, cap, 1.0f / cap);
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
 
 CGK_API int cgk_embed_sinusoid(const void* ids, const void* pos, const void* table, int table_fp32, float scale, const void* freq,
                                void* x, void* h, int h_fp32, int rows, int D, int vocab, void* stream) {

@@ -2,7 +2,7 @@
 // plain 16-byte loads, fp32 sums.  A tensor-core tile would compute 128 rows and stream the weights through a
 // quarter of the SMs; here every warp owns a few weight rows and keeps several loads in flight per lane.
 //   plain   one batch entry per blockIdx.y
-//   gated   W holds gate rows then up rows: out = silu(gate) * up, the feed-forward's first half in one kernel
+//   gated   W holds gate rows then up rows: out = silu(gate) * up (or relu), the feed-forward's first half in one kernel
 //   b_mn    W stored [k][n] (the latent image of a query: W_uk^T q per head)
 #include "../../include/cogito_kernels.h"
 #include "host_common.h"
@@ -31,7 +31,7 @@ struct SkinnyDev {
   const __nv_bfloat16* x; long long ldx, sx;
   const __nv_bfloat16* w; long long ldw, sw;
   void* out; long long ldo, so;
-  int out_fp32, M, N, K;
+  int out_fp32, M, N, K, relu;
 };
 
 // MT: rows of x held (M <= MT), RW: output columns per warp; GATED: each column needs weight rows n and N + n
@@ -91,7 +91,7 @@ skinny_kernel(const SkinnyDev a) {
     for (int m = 0; m < MT; ++m)
       if (lane == r * MT + m && n0 + r < a.N && m < a.M) {
         float v = acc[r][m];
-        if (GATED) v = v / (1.0f + expf(-v)) * acc[RW + r][m];
+        if (GATED) v = (a.relu ? fmaxf(v, 0.0f) : v / (1.0f + expf(-v))) * acc[RW + r][m];
         const long long o = blockIdx.y * a.so + m * a.ldo + n0 + r;
         if (a.out_fp32) reinterpret_cast<float*>(a.out)[o] = v;
         else reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16(v);
@@ -175,14 +175,14 @@ CGK_API int cgk_skinny_gemm(const void* x, long long ldx, long long sx, const vo
                             long long so, int out_fp32, int M, int N, int K, int batch, int mode, void* stream) {
   using namespace cgk;
   CGK_REQUIRE(x && w && out && M >= 0 && M <= 8 && N >= 0 && K > 0 && batch >= 1 && batch <= 65535, "cgk_skinny_gemm: 1 to 8 rows");
-  CGK_REQUIRE(mode >= 0 && mode <= 2 && (mode != 1 || batch == 1), "cgk_skinny_gemm: bad mode");
+  CGK_REQUIRE(mode >= 0 && mode <= 3 && ((mode & 1) == 0 || batch == 1), "cgk_skinny_gemm: bad mode");
   auto al = [](const void* p, long long ld, long long s) { return (((uintptr_t)p) & 15) == 0 && ld % 8 == 0 && s % 8 == 0; };
   CGK_REQUIRE(al(w, ldw, sw) && (mode == 2 ? N % 8 == 0 : (K % 8 == 0 && al(x, ldx, sx))), "cgk_skinny_gemm: rows must be 16-byte aligned");
   if (M == 0 || N == 0) return 0;
   int dev = 0;
   CGK_CUDA_CHECK(cudaGetDevice(&dev));
   const int sms = sm_count(dev);
-  SkinnyDev d{(const __nv_bfloat16*)x, ldx, sx, (const __nv_bfloat16*)w, ldw, sw, out, ldo, so, out_fp32, M, N, K};
+  SkinnyDev d{(const __nv_bfloat16*)x, ldx, sx, (const __nv_bfloat16*)w, ldw, sw, out, ldo, so, out_fp32, M, N, K, mode == 3};
   cudaStream_t st = (cudaStream_t)stream;
   switch (mode) {
     case 0:
@@ -191,6 +191,7 @@ CGK_API int cgk_skinny_gemm(const void* x, long long ldx, long long sx, const vo
       if (M <= 4) return launch_rw<4, false>(d, batch, sms, st);
       return launch_rw<8, false>(d, batch, sms, st);
     case 1:
+    case 3:
       if (M == 1) return launch_rw<1, true>(d, 1, sms, st);
       if (M == 2) return launch_rw<2, true>(d, 1, sms, st);
       if (M <= 4) return launch_rw<4, true>(d, 1, sms, st);

@@ -1,4 +1,4 @@
-// silu(gate) * up over bf16 rows [gate | up] of 2 F elements, F a multiple of 8: four rows at a time per CTA, so every
+// act(gate) * up (act: silu or relu) over bf16 rows [gate | up] of 2 F elements, F a multiple of 8: four rows at a time per CTA, so every
 // thread keeps eight 16-byte loads in flight.  blockIdx.y picks a range of columns (few long rows still fill the GPU).
 #pragma once
 #include "sm100.cuh"
@@ -7,7 +7,12 @@ namespace cgk {
 
 constexpr int SWIGLU_ROWS = 4;
 
-__device__ __forceinline__ void swiglu_rows_bf16(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act, long long rows, int F) {
+enum : int { GATED_SILU = 0, GATED_RELU = 1 };
+template <int ACT>
+__device__ __forceinline__ float gated_act(float x) { return ACT == GATED_RELU ? fmaxf(x, 0.0f) : silu_f(x); }
+
+template <int ACT = GATED_SILU>
+__device__ __forceinline__ void swiglu_rows_bf16(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act, long long ldo, long long rows, int F) {
   for (long long row0 = (long long)blockIdx.x * SWIGLU_ROWS; row0 < rows; row0 += (long long)gridDim.x * SWIGLU_ROWS) {
     const int f = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
     if (f < F) {
@@ -27,9 +32,9 @@ __device__ __forceinline__ void swiglu_rows_bf16(const __nv_bfloat16* __restrict
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const float2 a = unpack_bf16x2(gw[e]), b = unpack_bf16x2(uw[e]);
-          o[e] = pack_bf16x2(silu_f(a.x) * b.x, silu_f(a.y) * b.y);
+          o[e] = pack_bf16x2(gated_act<ACT>(a.x) * b.x, gated_act<ACT>(a.y) * b.y);
         }
-        *reinterpret_cast<uint4*>(act + (row0 + j) * F + f) = make_uint4(o[0], o[1], o[2], o[3]);
+        *reinterpret_cast<uint4*>(act + (row0 + j) * ldo + f) = make_uint4(o[0], o[1], o[2], o[3]);
       }
     }
   }

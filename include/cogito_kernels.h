@@ -193,6 +193,11 @@ typedef struct {
   int64_t dv_bs, dv_ts, dv_hs;
   float* delta;               /* scratch fp32 [B, Hq, Tq] */
   float* dq_accum;            /* scratch fp32 [B, Tq, Hq, D] */
+  /* forward only, zero for the plain form: */
+  int32_t block;              /* > 0: with causal, key k only if it lies in the query's block of that many keys (counted from key 0) */
+  int32_t sink;               /* 1: one is added to the softmax denominator (a key of score 0 without a value) */
+  const void* turn;           /* (cos, sin) fp32 [B * Tq][o_cols / 2][2]: output pairs (2i, 2i + 1) are turned back by these */
+  int32_t o_cols;             /* > 0: only the first o_cols elements of a head's result are stored (any strides and alignment) */
 } cgk_flash_args;
 
 int cgk_flash_forward(const cgk_flash_args* args, void* stream);
@@ -286,6 +291,17 @@ typedef struct {
   float eps;
 } cgk_stream_update_args;
 int cgk_stream_update(const cgk_stream_update_args* a, void* stream);
+/* x[t] = table[ids[t]] (ids given) or x[t] + mult * y[t] (y given) or unchanged;  r = x[t] / sqrt(mean(x[t]^2) + eps);
+ * h1[t] = r * w1, h2[t] = r * w2 (each may be null).  One pass for layers whose sublayers read one stream through norms of their own. */
+typedef struct {
+  const int64_t* ids; const void* table; const void* y; int64_t ldy;
+  const float* w1; const float* w2; float* x; void* h1; void* h2;
+  int32_t rows, D, vocab, table_fp32, y_fp32, h_fp32;
+  float mult, eps;
+} cgk_stream_norms_args;
+int cgk_stream_norms(const cgk_stream_norms_args* a, void* stream);
+/* x = cap * tanh(x / cap), fp32, in place. */
+int cgk_softcap(void* x, long long n, float cap, void* stream);
 /* out[i] = rms_norm(x[rows[i]]) * w  (rows int64, null = identity; n_rows rows exist). */
 int cgk_rms_rows(const void* x, const void* rows, int n_out, int n_rows, const void* w, void* out, int out_fp32, int D, float eps,
                  void* stream);
@@ -294,7 +310,8 @@ int cgk_gemm_f32(const void* A, const void* B, void* C, int M, int N, int K, int
                  long long sA, long long sB, long long sC, int b_mn, void* stream);
 
 /* Products with up to 8 rows (decoding), bf16 operands, fp32 sums: out[b, m, n] = sum_k x[b, m, k] W[b, n, k].
- * mode 0: plain; 1: gated, W holds N gate rows then N up rows and out = silu(gate) * up (batch 1); 2: W stored [K, N]. */
+ * mode 0: plain; 1: gated, W holds N gate rows then N up rows and out = silu(gate) * up (batch 1); 2: W stored [K, N];
+ * 3: gated with relu in the place of silu. */
 int cgk_skinny_gemm(const void* x, long long ldx, long long sx, const void* w, long long ldw, long long sw, void* out, long long ldo,
                     long long so, int out_fp32, int M, int N, int K, int batch, int mode, void* stream);
 
@@ -321,6 +338,55 @@ int cgk_latent_attention(const cgk_latent_args* a, const void* q, void* out, int
 int cgk_latent_attention_tc_ok(int R, int page_size, int heads);
 long long cgk_latent_attention_scratch_floats(int rows, int heads, int R, int splits);
 
+/* ---- Paged keys and values with rotary positions (csrc/kernels/kv_rows.cu) ---- */
+/* One layer's cache: k_pages[n_pages][kv_heads][page_size][ceil8(dim)], v_pages likewise with vdim, bf16 (fp32 with `fp32`),
+ * row tails zero; the tokens of a call: token t belongs to the sequence in slot[t] and stands at pos[t]. */
+typedef struct {
+  void* k_pages; void* v_pages;
+  const int32_t* page_table;         /* [slots][max_pages] */
+  const int32_t* slot; const int32_t* pos;
+  int32_t kv_heads, dim, vdim, page_size, max_pages, slots, n_pages, fp32;
+} cgk_kv_rows_args;
+/* cs[t][i] = (cos, sin) of pos[t] * freq[i]; freq fp64 [pairs], cs fp32 [rows][pairs][2]. */
+int cgk_rotary_angles(const void* pos, const void* freq, void* cs, int rows, int pairs, void* stream);
+/* q_out[t][h] = q[t][h] with its first `rot` elements turned pair by pair (2i, 2i + 1) by cs_k; keys likewise and values (RMS-normed
+ * over vdim with norm_v, turned by cs_v if given) go to the token's cache place and, if k_out / v_out are given, there too.
+ * q_out, k_out, v_out: [rows][heads][wide], tails zero.  k and v null: queries only. */
+typedef struct {
+  const void* q; const void* k; const void* v;
+  int64_t ldq, ldk, ldv;
+  const void* cs_k; const void* cs_v;
+  void* q_out; void* k_out; void* v_out;
+  int32_t heads, rot, wide, norm_v;
+  float eps;
+} cgk_kv_prep_args;
+int cgk_kv_rotate_append(const cgk_kv_rows_args* c, const cgk_kv_prep_args* a, int rows, void* stream);
+/* Keys and values of positions first .. first + len - 1 of `slot` -> [len][kv_heads][wide]. */
+int cgk_kv_gather(const cgk_kv_rows_args* c, int slot, int first, int len, int wide, void* k_out, void* v_out, void* stream);
+/* out[t][h] (rows ldo apart, heads vdim apart) = sum_j p_j v_j over the positions j <= pos[t] of the token's sequence - with block > 0
+ * only those of pos[t]'s block of that many positions - p the softmax of scale * q.k, with `sink` one added to its denominator;
+ * the sum is turned back by `turn` (cos, sin [rows][vdim / 2]) if given.  splits > 1: key ranges handled by separate CTAs. */
+int cgk_kv_rows_attention(const cgk_kv_rows_args* c, const void* q, long long ldq, int wide, void* out, long long ldo, const void* turn,
+                          int rows, int heads, float scale, int block, int sink, int splits, void* scratch, void* stream);
+long long cgk_kv_rows_scratch_floats(int rows, int heads, int vdim, int splits);
+
+/* ---- Linear recurrences with a decay per state row (csrc/kernels/linear_state.cu, linear_state_tc.cu) ---- */
+/* Per head: S = diag(a) S + k v^T, o = S^T q, out = rms(o) * w (* silu(gate)).  With y = z + bias:
+ * mode 0: a = low + (1 - low) sigmoid(y), k = 1 - a;  mode 1: a = sigmoid(y)^inv_tau, k given.  q enters as (silu of it with q_silu) * q_scale.
+ * state [slots][history][heads][D][V] fp32, the state after p tokens in entry p mod history; a sequence at position 0 starts from zeros.
+ * runs [n_runs][2]: first row and number of consecutive tokens of one sequence; null: every row is a run. */
+typedef struct {
+  const void* q; const void* k; const void* v; const void* gate; const float* z;
+  int64_t ldq, ldk, ldv, ldg, ldz;
+  const float* bias; const float* low; const float* w;
+  float* state;
+  void* out; int64_t ldo;
+  const int32_t* slot; const int32_t* pos; const int32_t* runs;
+  int32_t heads, D, V, history, slots, mode, q_silu, fp32;
+  float q_scale, inv_tau, eps;
+} cgk_linear_state_args;
+int cgk_linear_state(const cgk_linear_state_args* a, int n_runs, void* stream);
+
 /* ---- Mixture of experts (csrc/kernels/moe.cu) ---- */
 /* scores s = softmax(logits[t]); choice = s + correction; only outputs of the `keep` best of `groups` equal groups
  * (by largest choice score) can be chosen; idx = the `top` best choices, weight = their s over the sum.  row_of =
@@ -333,6 +399,8 @@ int cgk_moe_gather(const void* h, const void* idx, int pairs, int top, int exper
                    int max_rows, void* stream);
 /* g: A [rows][K] in expert order, B [experts][N][K], out bf16 or fp32 [rows][N]; g->M = allocated rows (a multiple of 128). */
 int cgk_gemm_grouped_bf16(const cgk_gemm_args* g, const int* tile_group, const int* tiles, void* stream);
+/* out[r] = act(gu[r][:F]) * gu[r][F:], rows of out ldo apart; dtype 0 fp32, 1 bf16; act 0 silu, 1 relu. */
+int cgk_gated_rows(int dtype, const void* gu, void* out, long long ldo, long long rows, int F, int act, void* stream);
 int cgk_swiglu_tiles(const void* gate_up, void* act, const void* tiles, int F, int max_tiles, void* stream);
 /* Expert products pair by pair: act [pairs][F] in the weights' type, y fp32 [pairs][D]; w_gate_up [experts][2F][D], w_down
  * [experts][D][F].  Pairs whose output is not an expert are left alone. */

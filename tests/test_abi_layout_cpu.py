@@ -11,13 +11,15 @@ ROOT = Path(__file__).resolve().parent.parent
 
 
 def _pairs():
-    from cogito_b200.ops import _lib, attention, stream
+    from cogito_b200.ops import _lib, attention, recurrence, stream
     from cogito_b200.parallel import data_parallel, tp_ops
-    from cogito_b200.serve import kv_cache
+    from cogito_b200.serve import hybrid_cache, kv_cache
     return [("cgk_gemm_args", _lib.GemmArgs), ("cgk_flash_args", attention.FlashArgs), ("cgk_ag_args", tp_ops.AgArgs),
             ("cgk_rs_args", tp_ops.RsArgs), ("cgk_dp_bucket_args", data_parallel.DpBucketArgs),
             ("cgk_dp_finish_args", data_parallel.DpFinishArgs), ("cgk_kv_args", kv_cache.KvArgs),
-            ("cgk_latent_args", kv_cache.LatentArgs), ("cgk_stream_update_args", stream.StreamUpdateArgs)]
+            ("cgk_latent_args", kv_cache.LatentArgs), ("cgk_stream_update_args", stream.StreamUpdateArgs),
+            ("cgk_stream_norms_args", stream.StreamNormsArgs), ("cgk_kv_rows_args", hybrid_cache.KvRowsArgs),
+            ("cgk_kv_prep_args", hybrid_cache.KvPrepArgs), ("cgk_linear_state_args", recurrence.LinearStateArgs)]
 
 
 @pytest.mark.skipif(shutil.which("gcc") is None and shutil.which("cc") is None, reason="needs a C compiler")
