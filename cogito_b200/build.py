@@ -101,7 +101,7 @@ def _build(sources: list[Path], headers: list[Path], out: Path, compiler: list[s
 # The kernels a layer-stack model is served with (serve.stack): enough for a checkout that only serves, in a
 # fraction of the time the whole library takes.
 SERVE_SOURCES = ("elementwise", "flash_fwd", "gemm_f32", "gemm_tcgen05", "host_common", "kv_rows", "latent_attn_tc", "latent_kv",
-                 "linear_state", "moe", "kv_attn_tc", "residual_stream", "serving", "skinny_gemm")
+                 "linear_state", "linear_state_tc", "moe", "kv_attn_tc", "residual_stream", "serving", "skinny_gemm")
 
 
 def build_serving_kernels(verbose: bool = False, out: Path | None = None) -> Path:

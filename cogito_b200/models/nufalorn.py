@@ -51,7 +51,7 @@ class NufalornConfig:
 
     @classmethod
     def from_dict(cls, d: dict, shapes: dict[str, tuple[int, ...]] | None = None) -> "NufalornConfig":
-        """shapes: the checkpoint's tensors; they give the one size that the dictionary does not have."""
+        """shapes: the checkpoint's tensors; they give the inner size of the gated decay (or the mixer's key ``a_rank``)."""
         layers = []
         for i, e in enumerate(d["layers"]):
             m, mlp, kind, rank = e["mixer"], e.get("mlp"), e["type"], 0
@@ -62,7 +62,7 @@ class NufalornConfig:
             elif kind in RECURRENT:
                 mixer = RecurrentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"]) if kind == "gla" else 1.0)
                 if kind == "gla":
-                    rank = int(shapes[f"l{i}.mix.a1"][0]) if shapes and f"l{i}.mix.a1" in shapes else int(m.get("a_rank", 16))
+                    rank = int(shapes[f"l{i}.mix.a1"][0]) if shapes and f"l{i}.mix.a1" in shapes else int(m["a_rank"])
             else:
                 raise ValueError(f"layer {i}: unknown mixer {kind!r}")
             layers.append(LayerSpec(kind, mixer, None if mlp is None else DenseSpec(int(mlp["ff"])), rank))
@@ -99,7 +99,7 @@ class NufalornConfig:
                 if s.kv_from is not None:
                     m["kv_from"] = s.kv_from
             elif l.kind == "gla":
-                m["tau"] = l.mixer.tau
+                m.update(tau=l.mixer.tau, a_rank=l.a_rank)
             out.append({"type": l.kind, "mixer": m, "mlp": None if l.mlp is None else {"kind": "dense", "ff": l.mlp.ff}})
         return {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.width, "residual_mult": self.residual_mult,
                 "logit_softcap": self.logit_softcap, "norm": {"eps": self.norm_eps}, "layers": out}

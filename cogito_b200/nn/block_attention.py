@@ -17,6 +17,7 @@ from ..ops import rotary
 from ..ops.attention import flash_forward
 from ..ops.linear import linear
 from .latent_attention import _frozen
+from .parallel_layer import rows_of_8
 
 
 @dataclass(frozen=True)
@@ -52,7 +53,7 @@ class BlockAttention(nn.Module):
         self.spec, self.eps = spec, eps
         self.own = spec.kv_from is None
         parts = [tensors["q"]] + ([tensors["k"], tensors["v"]] if self.own else [])
-        self.w_in = _frozen(torch.cat([p.to(device) for p in parts], 0).to(dtype).contiguous())
+        self.w_in = _frozen(rows_of_8(torch.cat([p.to(device) for p in parts], 0)).to(dtype).contiguous())
         wide = max(spec.dim, spec.vdim)
         # the flash kernel takes heads of 64 or 128 elements: shorter ones get zero columns (exact)
         self.prompt_form = dtype == torch.bfloat16 and wide <= 128
@@ -80,7 +81,7 @@ class BlockAttention(nn.Module):
         cs_v = None if self.freq_v is None else step_angles(batch, self.freq_v)
         segs = batch.prompts if self.prompt_form else ()
         split = batch.single_from if self.prompt_form else 0
-        k, v = (x[:, nq:nq + nk], x[:, nq + nk:]) if self.own else (None, None)
+        k, v = (x[:, nq:nq + nk], x[:, nq + nk:nq + nk + s.kv_heads * s.vdim]) if self.own else (None, None)
         first = {id(g): g.begin // s.block * s.block if s.block else 0 for g in segs}
         q, kc, vc = cache.rotate_append(layer, x[:, :nq], k, v, cs_k, cs_v, s.heads, self.wide, batch.slot, batch.pos,
                                         self.eps if s.norm_values else None, keep=any(first[id(g)] == g.begin for g in segs))

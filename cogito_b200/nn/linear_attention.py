@@ -14,6 +14,7 @@ from torch import nn
 from ..ops import recurrence as R
 from ..ops.linear import linear
 from .latent_attention import _frozen
+from .parallel_layer import rows_of_8
 
 
 @dataclass(frozen=True)
@@ -29,7 +30,8 @@ class _Recurrent(nn.Module):
         super().__init__()
         self.spec = spec
         self._t = {k: v.to(device) for k, v in tensors.items()}
-        self._put = lambda *names: _frozen(torch.cat([self._t[n] for n in names], 0).to(dtype).contiguous())
+        # rows of a product start on 16 bytes: its columns are filled up to a multiple of 8
+        self._put = lambda *names: _frozen(rows_of_8(torch.cat([self._t[n] for n in names], 0)).to(dtype).contiguous())
         self._vec = lambda name: _frozen(self._t[name].float().contiguous())
 
     def _loaded(self):
@@ -65,7 +67,8 @@ class GatedLinearAttention(_Recurrent):
         s = self.spec
         x = linear(h, self.w_in, out_dtype=h.dtype)
         q, k, v, g, u = self._columns(x, s.heads * s.dim, s.heads * s.dim, s.heads * s.vdim, s.heads * s.vdim, self.w_a2.shape[1])
-        return R.Operands(q, k, v, g, linear(u, self.w_a2, out_dtype=torch.float32), self.bias, None, self.norm)
+        z = linear(u, self.w_a2, out_dtype=torch.float32)[:, :s.heads * s.dim]
+        return R.Operands(q, k, v, g, z, self.bias, None, self.norm)
 
 
 class Hgrn2(_Recurrent):
@@ -81,4 +84,5 @@ class Hgrn2(_Recurrent):
     def operands(self, h):
         s = self.spec
         q, v = self._columns(linear(h, self.w_in, out_dtype=h.dtype), s.heads * s.dim, s.heads * s.vdim)
-        return R.Operands(q, None, v, None, linear(h, self.w_f, out_dtype=torch.float32), self.bias, self.low, self.norm)
+        z = linear(h, self.w_f, out_dtype=torch.float32)[:, :s.heads * s.dim]
+        return R.Operands(q, None, v, None, z, self.bias, self.low, self.norm)

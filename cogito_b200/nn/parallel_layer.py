@@ -17,6 +17,11 @@ def _ceil8(n: int) -> int:
     return (n + 7) // 8 * 8
 
 
+def rows_of_8(w: torch.Tensor) -> torch.Tensor:
+    """[n, K] with zero rows up to a multiple of 8."""
+    return torch.nn.functional.pad(w, (0, 0, 0, _ceil8(w.shape[0]) - w.shape[0]))
+
+
 class ParallelLayer(nn.Module):
     """mixer: a module with ``out_width`` that is called as mixer(h, batch, cache, layer, out); mlp: a ``GatedMLP`` or None;
     w_o: the mixer's output matrix [width, out_width]; norm1, norm2: fp32 norm weights (norm2 None without mlp)."""

@@ -22,7 +22,7 @@ if not _DEBUG and not _LIB_PATH.exists() and (_LIB_DIR / "libcogito_kernels_serv
 _lib = None
 # source files that carry index checks in the debug build (one recorded violation each)
 _BOUNDS_FILES = ("gemm_tcgen05", "softmax_ce", "serving", "elementwise", "flash_fwd", "flash_bwd", "residual_stream", "latent_kv",
-                 "latent_attn_tc", "moe", "kv_rows", "linear_state")
+                 "latent_attn_tc", "moe", "kv_rows", "linear_state", "linear_state_tc")
 
 
 class KernelError(RuntimeError):
@@ -123,6 +123,8 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_kv_gather": [vp, i, i, i, i, vp, vp, vp],
         "cgk_kv_rows_attention": [vp, vp, ll, i, vp, ll, vp, i, i, f, i, i, i, vp, vp],
         "cgk_linear_state": [vp, i, vp],
+        "cgk_linear_chunks": [vp, vp, i, vp, i, vp, vp],
+        "cgk_linear_chunks_ok": [i, i],
         "cgk_stream_norms": [vp, vp],
         "cgk_softcap": [vp, ll, f, vp],
         "cgk_gated_rows": [i, vp, vp, ll, ll, i, i, vp],
@@ -142,6 +144,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_int4_gemm_counters": [i, i],
         "cgk_latent_attention_scratch_floats": [i, i, i, i],
         "cgk_kv_rows_scratch_floats": [i, i, i, i],
+        "cgk_linear_chunks_scratch_floats": [i, i, i, i],
     }.items():
         fn = getattr(L, name, None)
         if fn is None:                              # a library built from part of the sources

@@ -104,15 +104,68 @@ def _args(rule, x, state, slot, pos, runs, out) -> LinearStateArgs:
     return a
 
 
+CHUNK = 64                  # tokens per step of the tensor-core form
+SMS = 148
+
+
+def stretches(counts: list[int], heads: int, first_rows: list[int]):
+    """Cuts runs of the given lengths into stretches that are handled side by side, whole chunks long.  The cut takes
+    the fewest chunks one after another: rounds of CTAs (one per stretch and head) times the stretch's chunks, and about
+    0.6 of that again for the pass that sums the stretches up, if any run is cut.
+    Returns (items [n][4], run_items [runs][2], whether a run is cut)."""
+    chunks = [-(-n // CHUNK) for n in counts]
+    best = None
+    for n in range(1, 33):
+        length = -(-max(chunks) // n)
+        items = sum(-(-c // length) for c in chunks)
+        cost = -(-items * heads // SMS) * length * (1.0 if items == len(chunks) else 1.6)
+        if best is None or cost < best[0]:
+            best = cost, length
+    size, items, run_items = best[1] * CHUNK, [], []
+    for r, (n, row) in enumerate(zip(counts, first_rows)):
+        run_items.append([len(items), -(-n // size)])
+        for at in range(0, n, size):
+            items.append([row + at, min(size, n - at), r, int(at + size >= n)])
+    return items, run_items, len(items) > len(counts)
+
+
+def _chunked(rule: StateRule, x: Operands) -> bool:
+    """Whether the tensor-core form takes these operands."""
+    if x.q.dtype != torch.bfloat16 or not _lib.lib().cgk_linear_chunks_ok(rule.dim, rule.vdim):
+        return False
+    return all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (x.q, x.k, x.v, x.gate, x.z))
+
+
+def _advance_chunks(a: LinearStateArgs, rule: StateRule, batch, device):
+    key = ("stretches", rule.heads)
+    if key not in batch.memo:
+        rows = [g.start + i * g.count for g in batch.prompts for i in range(g.sequences)]
+        items, run_items, cut = stretches([g.count for g in batch.prompts for _ in range(g.sequences)], rule.heads, rows)
+        flat = torch.tensor([v for t in items + run_items for v in t], dtype=torch.int32).to(device)
+        batch.memo[key] = flat, len(items), len(run_items), cut
+    flat, n, runs, cut = batch.memo[key]
+    L, scratch = _lib.lib(), None
+    if cut:
+        scratch = torch.empty(L.cgk_linear_chunks_scratch_floats(n, rule.heads, rule.dim, rule.vdim), dtype=torch.float32, device=device)
+    _lib.check(L.cgk_linear_chunks(ctypes.byref(a), flat.data_ptr(), n, flat[4 * n:].data_ptr(), runs, _lib.ptr(scratch), _lib.stream_ptr()),
+               "cgk_linear_chunks")
+    _lib.count_launch(3 if cut else 1)
+
+
 def advance(rule: StateRule, x: Operands, state, batch, out):
     """The recurrence over the runs of ``batch`` (slot, pos; runs int32 [n, 2]: first row and number of consecutive tokens of
-    one sequence, None: every row is a run).  state fp32 [slots, history, heads, dim, vdim]: the state after p tokens of a
-    sequence is entry p mod history of its slot; a sequence at position 0 starts from zeros.  ``out`` [N, heads * vdim] may
-    be a view with longer rows; returned."""
+    one sequence, None: every row is a run; prompts: the runs that come first and take the chunked form).  state fp32
+    [slots, history, heads, dim, vdim]: the state after p tokens of a sequence is entry p mod history of its slot; a
+    sequence at position 0 starts from zeros.  ``out`` [N, heads * vdim] may be a view with longer rows; returned."""
     slot, pos, runs = batch.slot, batch.pos, batch.runs
     if not x.q.is_cuda:
         return _advance_cpu(rule, x, state, slot, pos, runs, out)
-    a = _args(rule, x, state, slot, pos, runs, out)
-    _lib.check(_lib.lib().cgk_linear_state(ctypes.byref(a), x.q.shape[0] if runs is None else runs.shape[0], _lib.stream_ptr()), "cgk_linear_state")
-    _lib.count_launch()
+    if batch.prompts and _chunked(rule, x) and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0:
+        _advance_chunks(_args(rule, x, state, slot, pos, None, out), rule, batch, out.device)
+        runs = runs[sum(g.sequences for g in batch.prompts):]
+    n = x.q.shape[0] if runs is None else runs.shape[0]
+    if n:
+        a = _args(rule, x, state, slot, pos, runs, out)
+        _lib.check(_lib.lib().cgk_linear_state(ctypes.byref(a), n, _lib.stream_ptr()), "cgk_linear_state")
+        _lib.count_launch()
     return out

@@ -159,8 +159,8 @@ class HybridCache(PagedCache):
             for t in range(N):
                 p = int(pos[t])
                 lo = p // block * block if block else 0
-                k, v = (x.float().repeat_interleave(group, 1) for x in self.gather(layer, int(slot[t]), lo, p + 1 - lo, wide))
-                sc = torch.einsum("hd,khd->hk", q[t].float(), k) * scale
+                k, v = (x.float().repeat_interleave(group, 1) for x in self.gather(layer, int(slot[t]), lo, p + 1 - lo, max(wide, s.vdim)))
+                sc = torch.einsum("hd,khd->hk", q[t].float(), k[..., :wide]) * scale
                 if sink:
                     sc = torch.cat([sc, torch.zeros(H, 1)], 1)
                 o = torch.einsum("hk,khd->hd", torch.softmax(sc, -1)[:, :p + 1 - lo], v[..., :s.vdim])

@@ -1,0 +1,509 @@
+// Linear recurrences (linear_state.cuh) over prompt portions, 64 tokens at a time on the tcgen05 tensor cores.
+//
+// With b_t the logarithm of the decay since the start of a chunk (per state row), r its value in the chunk's middle,
+//     Q = q 2^(b - r),  K = k 2^(r - b),  A = tril(Q K^T),  O = A V + Q (2^r S),  S' = 2^(b_end - r) (2^r S + K^T V)
+// so a chunk takes four products.  The state stays in TMEM in fp32 from chunk to chunk (times a factor per row that is kept
+// beside it); every fp32 operand enters the tensor core as the sum of two bf16 numbers (three products for two such
+// operands, the smallest one is dropped), so the sums see 16 bits of each factor.  Where a decay is so strong that
+// the exponents could leave fp32's range, A is formed term by term with b_t - b_s <= 0, and Q and K take the
+// chunk's ends as their references.
+//
+// One CTA walks the chunks of one (stretch of a run, head).  A long run is cut into stretches that run side by side: a
+// first pass sums up what each stretch adds to the state, a second one turns that into the stretches' first states.
+#include "../../include/cogito_kernels.h"
+#include "host_common.h"
+#include "linear_state.cuh"
+#include "sm100.cuh"
+#include "typed_io.cuh"
+
+namespace cgk {
+namespace {
+
+constexpr int LC = 64, LC_THREADS = 512;
+constexpr float LC_LIMIT = 100.0f;                        // largest exponent (base 2) of a factor
+// shared memory: operand tiles of 128-byte rows in blocks of 64 columns (bytes)
+constexpr uint32_t T_K = 0, T_V = 32768, T_Q = 49152, T_A = 81920, T_S = 98304, T_END = 163840;
+constexpr uint32_t T_END_SUM = T_Q;                       // the summing pass has K and V only
+constexpr uint32_t T_SPLIT = 16384;                       // high part -> low part of Q and K
+constexpr uint32_t LC_MISC = (8 * 128 + 4 * 128 + 4 * LC) * 4 + 64;
+constexpr uint32_t TM_S = 0, TM_O = 128, TM_A = 256;      // TMEM columns
+
+struct ChunksDev {
+  LinStateDev a;
+  const int* items;          // [n_items][4]: first row, tokens, run, last stretch of the run
+  float* start;              // [n_items][heads][D][V]: sums, then first states; null: every run is one stretch
+  float* total;              // [n_items][heads][D]: logarithm (base 2) of a stretch's whole decay
+  int* status;
+};
+
+__device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x0, x1);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(x0 - h.x, x1 - h.y);
+}
+// byte offset of a 4-byte pair of columns in a tile with `rows` rows per block
+__device__ __forceinline__ uint32_t pair_at(int row, int col, int rows) {
+  return (col >> 6) * (rows * 128) + sw128_offset(row, (col & 63) >> 3) + (col & 7) * 2;
+}
+
+template <bool OUT>
+__global__ void __launch_bounds__(LC_THREADS, OUT ? 1 : 2)
+linear_chunks_kernel(const ChunksDev c) {
+  const LinStateDev& a = c.a;
+  extern __shared__ uint8_t lc_raw[];
+  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lc_raw) + 1023) & ~uintptr_t(1023));
+  const uint32_t sb = smem_u32(sm);
+  constexpr uint32_t END = OUT ? T_END : T_END_SUM;
+  float* part = reinterpret_cast<float*>(sm + END);       // [8][128] decay of eight tokens
+  float* rq = part + 8 * 128;                             // [128] references of Q and K, pending factor, decay of all chunks
+  float* rk = rq + 128;
+  float* pend = rk + 128;
+  float* tot = pend + 128;
+  float* red = tot + 128;                                 // [4][64]
+  uint32_t* bars = reinterpret_cast<uint32_t*>(red + 4 * LC);
+  const uint32_t bar_a = smem_u32(bars), bar_o = bar_a + 8, bar_s = bar_a + 16;
+  volatile uint32_t* tmem_slot = bars + 6;
+  volatile int* dead = reinterpret_cast<volatile int*>(bars + 7);
+  volatile int* go = reinterpret_cast<volatile int*>(bars + 8);          // one word per barrier
+
+  const int* item = c.items + 4 * blockIdx.y;
+  const int row0 = item[0], count = item[1], last = item[3], h = blockIdx.x;
+  if (!OUT && last) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3, cg = warp >> 2;
+  const int D = a.D, V = a.V;
+  constexpr uint32_t COLS = OUT ? 512 : 128;
+
+  if (tid == 0) {
+    mbar_init(bar_a, 1);
+    mbar_init(bar_o, 1);
+    mbar_init(bar_s, 1);
+    *dead = 0;
+    mbar_fence_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(smem_u32((const void*)tmem_slot), COLS);
+    tmem_relinquish();
+  }
+  for (uint32_t i = tid; i < END / 16; i += LC_THREADS) reinterpret_cast<uint4*>(sm)[i] = make_uint4(0, 0, 0, 0);
+  if (tid < 128) { pend[tid] = 0.0f; tot[tid] = 0.0f; }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const uint32_t lanes = (uint32_t)(quad * 32) << 16;
+
+  // first state -> TMEM: lane = state row, this warp's 32 columns
+  const int srow = quad * 32 + lane;
+  const int p0 = a.pos[row0];
+  const long long slot = CGK_IDX(a.slot[row0], a.slots);
+  {
+    const float* src = nullptr;
+    if (OUT && c.start) src = c.start + ((long long)blockIdx.y * a.heads + h) * D * V;
+    else if (OUT && p0 > 0) src = a.state + ((slot * a.history + p0 % a.history) * a.heads + h) * (long long)D * V;
+    uint32_t r[32];
+#pragma unroll
+    for (int j = 0; j < 32; j += 4) {
+      float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if (src && srow < D && cg * 32 + j < V) ldv<4>(src + (long long)srow * V + cg * 32 + j, v);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) r[j + e] = __float_as_uint(v[e]);
+    }
+    tmem_st32(tmem + TM_S + lanes + cg * 32, r);
+    tmem_st_wait();
+  }
+
+  const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(a.q) + (long long)row0 * a.ldq + h * D;
+  const __nv_bfloat16* kp = a.k ? reinterpret_cast<const __nv_bfloat16*>(a.k) + (long long)row0 * a.ldk + h * D : nullptr;
+  const __nv_bfloat16* vp = reinterpret_cast<const __nv_bfloat16*>(a.v) + (long long)row0 * a.ldv + h * V;
+  const float* zp = a.z + (long long)row0 * a.ldz + h * D;
+  const int ch = (tid & 63) * 2, tg = tid >> 6;           // two state rows, eight tokens
+  const bool mine = ch < D;
+  const int ksteps = (D + 15) / 16, n_chunks = (count + LC - 1) / LC;
+  bool ok = true;
+
+  for (int n = 0; n < n_chunks && ok; ++n) {
+    const int t0 = n * LC, left = min(LC, count - t0);
+    // ---- decays, their sums, operands
+    float b[8][2], kv[8][2], qv[8][2];
+    float sum0 = 0.0f, sum1 = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int t = tg * 8 + i;
+      float g0 = 0.0f, g1 = 0.0f;
+      kv[i][0] = kv[i][1] = qv[i][0] = qv[i][1] = 0.0f;
+      if (mine && t < left) {
+        const float2 z = *reinterpret_cast<const float2*>(zp + (long long)(t0 + t) * a.ldz + ch);
+        g0 = lin_decay(a, z.x, h * D + ch, &kv[i][0]) * 1.4426950408889634f;
+        g1 = lin_decay(a, z.y, h * D + ch + 1, &kv[i][1]) * 1.4426950408889634f;
+        if (kp) {
+          const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(kp + (long long)(t0 + t) * a.ldk + ch));
+          kv[i][0] = k.x;
+          kv[i][1] = k.y;
+        }
+        if (OUT) {
+          const float2 q = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(qp + (long long)(t0 + t) * a.ldq + ch));
+          qv[i][0] = lin_query(a, q.x);
+          qv[i][1] = lin_query(a, q.y);
+        }
+      }
+      sum0 += g0;
+      sum1 += g1;
+      b[i][0] = sum0;
+      b[i][1] = sum1;
+    }
+    *reinterpret_cast<float2*>(part + tg * 128 + ch) = make_float2(sum0, sum1);
+    if (n > 0) {                                          // the previous chunk's products are done with the tiles and the state
+      if (tid == 0) go[0] = mbar_wait(bar_s, (n - 1) & 1, dead, c.status, 802);
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (n > 0 && !go[0]) { ok = false; break; }
+    float before[2] = {0.0f, 0.0f}, mid[2] = {0.0f, 0.0f}, end[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int g = 0; g < 8; ++g) {
+      const float2 s = *reinterpret_cast<const float2*>(part + g * 128 + ch);
+      if (g == tg) { before[0] = end[0]; before[1] = end[1]; }
+      end[0] += s.x;
+      end[1] += s.y;
+      if (g == 3) { mid[0] = end[0]; mid[1] = end[1]; }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { b[i][0] += before[0]; b[i][1] += before[1]; }
+    bool far = false;
+    if (OUT) {
+      const bool mine_far = fmaxf(-mid[0], -mid[1]) > LC_LIMIT || fmaxf(mid[0] - end[0], mid[1] - end[1]) > LC_LIMIT;
+      far = __syncthreads_or(mine_far) != 0;
+    }
+    float am[8];                                          // `far`: this thread's part of A, row tid / 8, columns 8 (tid % 8) ..
+    if (far) {
+      float* fb = reinterpret_cast<float*>(sm + T_S);
+      float* fq = fb + LC * 128;
+      float* fk = reinterpret_cast<float*>(sm + T_K);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int at = (tg * 8 + i) * 128 + ch;
+        *reinterpret_cast<float2*>(fb + at) = make_float2(b[i][0], b[i][1]);
+        *reinterpret_cast<float2*>(fq + at) = make_float2(qv[i][0], qv[i][1]);
+        *reinterpret_cast<float2*>(fk + at) = make_float2(kv[i][0], kv[i][1]);
+      }
+      __syncthreads();
+      const int t = tid >> 3, s0 = (tid & 7) * 8;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        float s = 0.0f;
+        if (s0 + j <= t)
+          for (int e = 0; e < D; ++e) s = fmaf(fq[t * 128 + e] * fk[(s0 + j) * 128 + e], exp2f(fb[t * 128 + e] - fb[(s0 + j) * 128 + e]), s);
+        am[j] = s;
+      }
+      __syncthreads();
+    }
+    const float ref_q[2] = {far ? 0.0f : mid[0], far ? 0.0f : mid[1]};
+    const float ref_k[2] = {far || !OUT ? end[0] : mid[0], far || !OUT ? end[1] : mid[1]};
+    if (tg == 0) {
+      rq[ch] = ref_q[0]; rq[ch + 1] = ref_q[1];
+      rk[ch] = ref_k[0]; rk[ch + 1] = ref_k[1];
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int t = tg * 8 + i;
+      const uint32_t at = pair_at(t, ch, LC);
+      uint32_t hi, lo;
+      split2(kv[i][0] * fast_exp2(ref_k[0] - b[i][0]), kv[i][1] * fast_exp2(ref_k[1] - b[i][1]), hi, lo);
+      *reinterpret_cast<uint32_t*>(sm + T_K + at) = hi;
+      *reinterpret_cast<uint32_t*>(sm + T_K + T_SPLIT + at) = lo;
+      if (OUT) {
+        split2(qv[i][0] * fast_exp2(b[i][0] - ref_q[0]), qv[i][1] * fast_exp2(b[i][1] - ref_q[1]), hi, lo);
+        *reinterpret_cast<uint32_t*>(sm + T_Q + at) = hi;
+        *reinterpret_cast<uint32_t*>(sm + T_Q + T_SPLIT + at) = lo;
+      }
+    }
+    for (int i = tid; i < LC * (V / 8); i += LC_THREADS) {
+      const int t = i / (V / 8), col = (i - t * (V / 8)) * 8;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (t < left) v = *reinterpret_cast<const uint4*>(vp + (long long)(t0 + t) * a.ldv + col);
+      *reinterpret_cast<uint4*>(sm + T_V + pair_at(t, col, LC)) = v;
+    }
+    if (n + 1 < n_chunks) {                               // the next chunk's rows on their way to L2
+      const int t = t0 + LC + (tid >> 3), part8 = (tid & 7);
+      if (t < count) {
+        const char* pz = reinterpret_cast<const char*>(zp + (long long)t * a.ldz) + part8 * 64;
+        if (part8 * 16 < D) asm volatile("prefetch.global.L2 [%0];" ::"l"(pz));
+        if (part8 * 32 < D && part8 < 4) {
+          if (OUT) asm volatile("prefetch.global.L2 [%0];" ::"l"(qp + (long long)t * a.ldq + part8 * 32));
+          if (kp) asm volatile("prefetch.global.L2 [%0];" ::"l"(kp + (long long)t * a.ldk + part8 * 32));
+        }
+        if (part8 >= 4 && (part8 - 4) * 32 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(vp + (long long)t * a.ldv + (part8 - 4) * 32));
+      }
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+
+    if (OUT && tid == 0 && !far) {
+      const uint32_t id = make_idesc_bf16(128, LC, 0, 0);  // rows 64 .. 127 are not used
+#pragma unroll 1
+      for (int part3 = 0; part3 < 3; ++part3) {
+        const uint32_t q = sb + T_Q + (part3 == 2 ? T_SPLIT : 0), k = sb + T_K + (part3 == 1 ? T_SPLIT : 0);
+        for (int kk = 0; kk < ksteps; ++kk)
+          umma_f16(tmem + TM_A, make_smem_desc_sw128(q + (kk >> 2) * (LC * 128) + (kk & 3) * 32, 16, 1024),
+                   make_smem_desc_sw128(k + (kk >> 2) * (LC * 128) + (kk & 3) * 32, 16, 1024), id, (part3 | kk) != 0);
+      }
+      umma_commit(bar_a);
+    }
+    // ---- state: operand of the product with Q, and the sum that K^T V is added to
+    {
+      uint32_t r[32];
+      __syncwarp();
+      tmem_ld32(tmem + TM_S + lanes + cg * 32, r);
+      tmem_ld_wait();
+      const float f = exp2f(pend[srow]), fq = exp2f(rq[srow]), fk = exp2f(rk[srow]);
+#pragma unroll
+      for (int j = 0; j < 32; j += 8) {
+        float s[8];
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          s[e] = __uint_as_float(r[j + e]) * f;
+          r[j + e] = __float_as_uint(s[e] * fk);
+          s[e] *= fq;
+        }
+        if (OUT) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) split2(s[2 * e], s[2 * e + 1], hi[e], lo[e]);
+          const uint32_t at = T_S + pair_at(srow, cg * 32 + j, 128);
+          *reinterpret_cast<uint4*>(sm + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(sm + at + 32768) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
+      }
+      __syncwarp();
+      tmem_st32(tmem + TM_S + lanes + cg * 32, r);
+      tmem_st_wait();
+    }
+    if (OUT) {
+      if (tid == 0 && !far) go[1] = mbar_wait(bar_a, n & 1, dead, c.status, 800);
+      if (tid == 0 && far) { mbar_arrive(bar_a); go[1] = 1; }
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (OUT && !go[1]) { ok = false; break; }
+    // every thread has read the references: the pending factor of the next chunk
+    if (tg == 0) {
+      pend[ch] = end[0] - ref_k[0];
+      pend[ch + 1] = end[1] - ref_k[1];
+      tot[ch] += end[0];
+      tot[ch + 1] += end[1];
+    }
+    if (OUT) {
+      // ---- A, lower triangle, as two bf16 parts
+      if (far) {
+        const int t = tid >> 3, s0 = (tid & 7) * 8;
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split2(am[2 * e], am[2 * e + 1], hi[e], lo[e]);
+        const uint32_t at = T_A + sw128_offset(t, s0 >> 3);
+        *reinterpret_cast<uint4*>(sm + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(sm + at + 8192) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      } else if (quad < 2) {
+        const int t = quad * 32 + lane;
+        uint32_t r[16];
+        __syncwarp();
+        tmem_ld16(tmem + TM_A + lanes + cg * 16, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 16; j += 8) {
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int s = cg * 16 + j + 2 * e;
+            split2(s <= t ? __uint_as_float(r[j + 2 * e]) : 0.0f, s + 1 <= t ? __uint_as_float(r[j + 2 * e + 1]) : 0.0f, hi[e], lo[e]);
+          }
+          const uint32_t at = T_A + sw128_offset(t, (cg * 16 + j) >> 3);
+          *reinterpret_cast<uint4*>(sm + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(sm + at + 8192) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      __syncthreads();
+      tc_fence_after();
+    }
+    if (tid == 0) {
+      const uint32_t v = sb + T_V;
+      if (OUT) {
+        const uint32_t id = make_idesc_bf16(128, 128, 0, 1);
+#pragma unroll 1
+        for (int part3 = 0; part3 < 3; ++part3) {
+          const uint32_t q = sb + T_Q + (part3 == 2 ? T_SPLIT : 0), s = sb + T_S + (part3 == 1 ? 32768 : 0);
+          for (int kk = 0; kk < ksteps; ++kk)
+            umma_f16(tmem + TM_O, make_smem_desc_sw128(q + (kk >> 2) * (LC * 128) + (kk & 3) * 32, 16, 1024),
+                     make_smem_desc_sw128(s + kk * 2048, 16384, 1024), id, (part3 | kk) != 0);
+        }
+#pragma unroll 1
+        for (int part2 = 0; part2 < 2; ++part2)
+          for (int kk = 0; kk < LC / 16; ++kk)
+            umma_f16(tmem + TM_O, make_smem_desc_sw128(sb + T_A + part2 * 8192 + kk * 32, 16, 1024), make_smem_desc_sw128(v + kk * 2048, 8192, 1024), id, 1);
+        umma_commit(bar_o);
+      }
+      const uint32_t id = make_idesc_bf16(128, 128, 1, 1);
+#pragma unroll 1
+      for (int part2 = 0; part2 < 2; ++part2)
+        for (int kk = 0; kk < LC / 16; ++kk)
+          umma_f16(tmem + TM_S, make_smem_desc_sw128(sb + T_K + part2 * T_SPLIT + kk * 2048, 8192, 1024), make_smem_desc_sw128(v + kk * 2048, 8192, 1024), id, 1);
+      umma_commit(bar_s);
+      if (OUT) go[2] = mbar_wait(bar_o, n & 1, dead, c.status, 801);
+    }
+    if (OUT) {
+      __syncthreads();
+      tc_fence_after();
+      if (!go[2]) { ok = false; break; }
+      // ---- result: lane = token, this warp's 32 columns; norm over the head, gate
+      if (quad < 2) {
+        const int t = quad * 32 + lane;
+        uint32_t r[32];
+        __syncwarp();
+        tmem_ld32(tmem + TM_O + lanes + cg * 32, r);
+        tmem_ld_wait();
+        float ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) ss = fmaf(__uint_as_float(r[j]), __uint_as_float(r[j]), ss);
+        red[cg * LC + t] = ss;
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (t < left) {
+          const float rs = 1.0f / sqrtf((red[t] + red[LC + t] + red[2 * LC + t] + red[3 * LC + t]) / V + a.eps);
+          const long long row = row0 + t0 + t;
+          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(a.out) + row * a.ldo + (long long)h * V + cg * 32;
+          const __nv_bfloat16* gp = a.gate ? reinterpret_cast<const __nv_bfloat16*>(a.gate) + row * a.ldg + (long long)h * V + cg * 32 : nullptr;
+#pragma unroll
+          for (int j = 0; j < 32; j += 8) {
+            if (cg * 32 + j >= V) continue;
+            float x[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(r[j + e]) * rs * a.w[cg * 32 + j + e];
+            if (gp) {
+              const uint4 g = *reinterpret_cast<const uint4*>(gp + j);
+              const uint32_t gu[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float2 f = unpack_bf16x2(gu[e]);
+                x[2 * e] *= silu_f(f.x);
+                x[2 * e + 1] *= silu_f(f.y);
+              }
+            }
+            *reinterpret_cast<uint4*>(o + j) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+          }
+        }
+      }
+    }
+  }
+  // ---- last state: to the cache, or as the stretch's sum
+  if (ok && n_chunks > 0) {
+    if (tid == 0) go[3] = mbar_wait(bar_s, (n_chunks - 1) & 1, dead, c.status, 803);
+    __syncthreads();
+    tc_fence_after();
+    ok = go[3] != 0;
+  }
+  if (ok && (!OUT || last)) {
+    uint32_t r[32];
+    __syncwarp();
+    tmem_ld32(tmem + TM_S + lanes + cg * 32, r);
+    tmem_ld_wait();
+    const float f = exp2f(pend[srow]);
+    float* dst = OUT ? a.state + ((slot * a.history + (p0 + count) % a.history) * a.heads + h) * (long long)D * V
+                     : c.start + ((long long)blockIdx.y * a.heads + h) * D * V;
+    if (srow < D) {
+#pragma unroll
+      for (int j = 0; j < 32; j += 4)
+        if (cg * 32 + j < V) {
+          const float v[4] = {__uint_as_float(r[j]) * f, __uint_as_float(r[j + 1]) * f, __uint_as_float(r[j + 2]) * f, __uint_as_float(r[j + 3]) * f};
+          stv<4>(dst + (long long)srow * V + cg * 32 + j, v);
+        }
+    }
+    if (!OUT && tid < D) c.total[((long long)blockIdx.y * a.heads + h) * D + tid] = tot[tid];
+  }
+  if (*dead) __nanosleep(100000);
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, COLS);
+  }
+}
+
+// Sums of a run's stretches -> their first states.  grid (state elements / 1024, heads, runs); four columns per thread.
+__global__ void __launch_bounds__(256)
+linear_starts_kernel(const ChunksDev c, const int* __restrict__ run_items) {
+  const LinStateDev& a = c.a;
+  const int e = (blockIdx.x * 256 + threadIdx.x) * 4, h = blockIdx.y, n0 = run_items[2 * blockIdx.z], n = run_items[2 * blockIdx.z + 1];
+  const int size = a.D * a.V, row = c.items[4 * n0], p0 = a.pos[row], d = e / a.V;
+  if (e >= size) return;
+  float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  if (p0 > 0) ldv<4>(a.state + ((CGK_IDX(a.slot[row], a.slots) * a.history + p0 % a.history) * a.heads + h) * (long long)size + e, s);
+  const long long step = (long long)a.heads * size;
+  float* at = c.start + ((long long)n0 * a.heads + h) * size + e;
+  const float* tot = c.total + ((long long)n0 * a.heads + h) * a.D + d;
+  float next[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  if (n > 1) ldv<4>(at, next);
+  for (int j = 0; j < n; ++j) {
+    const float add[4] = {next[0], next[1], next[2], next[3]};
+    if (j + 2 < n) ldv<4>(at + (j + 1) * step, next);
+    stv<4>(at + j * step, s);
+    if (j + 1 < n) {
+      const float f = exp2f(tot[(long long)j * a.heads * a.D]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[i] = fmaf(f, s[i], add[i]);
+    }
+  }
+}
+
+}  // namespace
+}  // namespace cgk
+
+using namespace cgk;
+
+CGK_API int cgk_linear_chunks_ok(int D, int V) { return D % 8 == 0 && V % 8 == 0 && D > 0 && V > 0 && D <= 128 && V <= 128; }
+
+CGK_API long long cgk_linear_chunks_scratch_floats(int n_items, int heads, int D, int V) { return (long long)n_items * heads * D * (V + 1); }
+
+CGK_API int cgk_linear_chunks(const cgk_linear_state_args* pa, const int* items, int n_items, const int* run_items, int n_runs, void* scratch,
+                              void* stream) {
+  CGK_REQUIRE(pa && items && n_items >= 0 && (!scratch || (run_items && n_runs > 0)), "cgk_linear_chunks: bad arguments");
+  const cgk_linear_state_args& a = *pa;
+  CGK_REQUIRE(a.q && a.v && a.z && a.bias && a.w && a.state && a.out && a.slot && a.pos && a.heads > 0 && a.history > 0 && a.slots > 0 && !a.fp32,
+              "cgk_linear_chunks: bad arguments");
+  CGK_REQUIRE(a.mode == GATE_BOUNDED ? (a.low && !a.k) : (a.mode == GATE_ROOT && a.k), "cgk_linear_chunks: the gate's operands do not fit its kind");
+  auto al = [](const void* p, long long ld) { return (((uintptr_t)p) & 15) == 0 && ld % 8 == 0; };
+  CGK_REQUIRE(cgk_linear_chunks_ok(a.D, a.V) && al(a.q, a.ldq) && al(a.k, a.k ? a.ldk : 0) && al(a.v, a.ldv) && al(a.gate, a.gate ? a.ldg : 0) &&
+              al(a.z, a.ldz) && al(a.out, a.ldo) && al(a.state, 0) && al(scratch, 0), "cgk_linear_chunks: sizes or alignment not supported");
+  CGK_REQUIRE(n_items <= 65535 && n_runs <= 65535, "cgk_linear_chunks: too many stretches in one call");
+  if (n_items == 0) return 0;
+  int dev = 0;
+  CGK_CUDA_CHECK(cudaGetDevice(&dev));
+  ChunksDev d;
+  d.a = LinStateDev{a.q, a.k, a.v, a.gate, a.z, a.ldq, a.ldk, a.ldv, a.ldg, a.ldz, a.bias, a.low, a.w, a.state, a.out, a.ldo, a.slot, a.pos, nullptr,
+                    a.heads, a.D, a.V, a.history, a.slots, a.mode, a.q_silu, a.q_scale, a.inv_tau, a.eps};
+  d.items = items;
+  d.start = (float*)scratch;
+  d.total = scratch ? (float*)scratch + (long long)n_items * a.heads * a.D * a.V : nullptr;
+  d.status = device_status(dev);
+  cudaStream_t st = (cudaStream_t)stream;
+  const dim3 grid(a.heads, n_items);
+  if (scratch) {
+    const int smem = T_END_SUM + LC_MISC + 1024;
+    CGK_CUDA_CHECK(cudaFuncSetAttribute(linear_chunks_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    linear_chunks_kernel<false><<<grid, LC_THREADS, smem, st>>>(d);
+    CGK_LAUNCH_CHECK();
+    linear_starts_kernel<<<dim3((a.D * a.V / 4 + 255) / 256, a.heads, n_runs), 256, 0, st>>>(d, run_items);
+    CGK_LAUNCH_CHECK();
+  }
+  const int smem = T_END + LC_MISC + 1024;
+  CGK_CUDA_CHECK(cudaFuncSetAttribute(linear_chunks_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  linear_chunks_kernel<true><<<grid, LC_THREADS, smem, st>>>(d);
+  CGK_LAUNCH_CHECK();
+  return 0;
+}
+
+CGK_BOUNDS_READER(linear_state_tc)
