@@ -9,7 +9,7 @@ Config (the reference's GPT-2-small line): 12 layers, d_model 768, 12 heads, MLP
 tensor parallel over the N GPUs (TP = N), so the total work is fixed ("strong").
 Synthetic data: token ids uniform over the vocabulary, weights N(0, 0.02).
 
-`--workload surelorn` measures the Surelorn serving path instead (benchmarks/surelorn.py).
+`--workload surelorn` and `--workload nufalorn` measure those serving paths instead (benchmarks/surelorn.py, nufalorn.py).
 
 Prints ONE JSON line on rank 0.  `value` is device-timed (CUDA events around
 exactly K steps, max over ranks) with the batch already on the device; `e2e` times
@@ -68,9 +68,9 @@ def parse():
                     help="on one GPU, also run the INT4 speculative-decoding configuration (Llama-7B shape, batch 16, "
                          "512-token prompts, 256 new tokens, gamma 4) as a child process after the training "
                          "measurements and report it under \"int4_spec_decode\" (auto = on)")
-    ap.add_argument("--workload", default="gpt2", choices=["gpt2", "surelorn"],
+    ap.add_argument("--workload", default="gpt2", choices=["gpt2", "surelorn", "nufalorn"],
                     help="gpt2: the headline training benchmark; surelorn: prompt and decode throughput of that model beside "
-                         "Llama at equal size (one GPU, --steps timed calls each; benchmarks/surelorn.py)")
+                         "Llama at equal size; nufalorn: that model beside Surelorn and Llama (one GPU, --steps timed calls each)")
     ap.add_argument("--timeline", default="", help="after the timed regions, trace two more steps and write the device "
                     "time per kernel name (rank 0) to this JSON file; not part of any reported number")
     args = ap.parse_args()
@@ -203,22 +203,22 @@ def kernel_timeline(step, path, rank, barrier, steps=2):
                    "last_step_launches": seq}, f, indent=1)
 
 
-def surelorn_workload(args):
-    """One JSON line: value = decode tokens/s of the larger dense Surelorn at batch 64, everything else beside it."""
-    import torch
+def serving_workload(args, name, kind):
+    """One JSON line: value = decode tokens/s of the larger model at batch 64, everything else beside it."""
+    import importlib
     here = os.path.dirname(os.path.abspath(__file__))
     sys.path[:0] = [here, os.path.join(here, "benchmarks")]
-    import surelorn
+    mod = importlib.import_module(name)
     from cogito_b200.ops import _lib
     sampler = ClockSampler(0)
     sampler.start()
     _lib.reset_launches()
-    rec = surelorn.run(iters=args.steps)
+    rec = mod.run(iters=args.steps)
     big = rec["sizes"][-1]
-    dec = big["model"]["surelorn_dense"]["decode_64"]
+    dec = big["model"][kind]["decode_64"]
     rec.update(value=dec["tok_per_s"], unit="tokens/s", n_gpus=1, steps=args.steps, warmup=max(args.warmup, 3), ms_per_step=dec["ms"],
                higher_is_better=True, vs_baseline=None, impl="cogito", clocks=sampler.stop(), gpu_launches=_lib.launches(),
-               config={"model": f"surelorn dense, width {big['width']}", "batch": 64, "context": surelorn.CONTEXT})
+               config={"model": f"{kind.replace('_', ' ')}, width {big['width']}", "batch": 64, "context": mod.CONTEXT})
     print(json.dumps(rec), flush=True)
     return 0
 
@@ -229,8 +229,8 @@ def main():
         print(json.dumps({"impl": "reference", "unavailable": REF_UNAVAILABLE}))
         return 0
 
-    if args.workload == "surelorn":
-        return surelorn_workload(args)
+    if args.workload != "gpt2":
+        return serving_workload(args, args.workload, {"surelorn": "surelorn_dense", "nufalorn": "nufalorn"}[args.workload])
 
     import torch
     import torch.distributed as dist

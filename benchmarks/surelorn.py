@@ -67,7 +67,7 @@ def _graph(fn):
     return g.replay
 
 
-def model_part(width, iters=10, prompts=((1, 2048), (4, 2048)), batches=(1, 16, 64)):
+def model_part(width, iters=10, prompts=((1, 2048), (4, 2048)), batches=(1, 16, 64), kinds=("dense", "mixture")):
     """Every timed region streams more weights than L2 holds."""
     from cogito_b200.models.llama import Llama, LlamaConfig
     from cogito_b200.models.surelorn import Surelorn, random_tensors
@@ -76,7 +76,7 @@ def model_part(width, iters=10, prompts=((1, 2048), (4, 2048)), batches=(1, 16, 
     s = SIZES[width]
     dev = torch.device("cuda")
     out = {"width": width, **{k: s[k] for k in ("heads", "layers", "ff", "kv_rank")}, "context": CONTEXT}
-    for kind in ("dense", "mixture"):
+    for kind in kinds:
         cfg = surelorn_config(width, s, kind == "mixture")
         model = Surelorn(cfg, random_tensors(cfg, 0, dev), dev, BF)
         rec = {"params": model.num_params()}
