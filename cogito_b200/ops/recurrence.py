@@ -109,16 +109,16 @@ SMS = 148
 
 
 def stretches(counts: list[int], heads: int, first_rows: list[int]):
-    """Cuts runs of the given lengths into stretches that are handled side by side, whole chunks long.  The cut takes
-    the fewest chunks one after another: rounds of CTAs (one per stretch and head) times the stretch's chunks, and about
-    0.6 of that again for the pass that sums the stretches up, if any run is cut.
+    """Cuts runs of the given lengths into stretches that are handled side by side, whole chunks long.  The cut costs the
+    least time by this count: rounds of CTAs (one per stretch and head) times the stretch's chunks and one more for a
+    CTA's start and end; summing the stretches up, needed if any run is cut, takes about 0.4 of that again.
     Returns (items [n][4], run_items [runs][2], whether a run is cut)."""
     chunks = [-(-n // CHUNK) for n in counts]
     best = None
     for n in range(1, 33):
         length = -(-max(chunks) // n)
         items = sum(-(-c // length) for c in chunks)
-        cost = -(-items * heads // SMS) * length * (1.0 if items == len(chunks) else 1.6)
+        cost = -(-items * heads // SMS) * (length + 1) * (1.0 if items == len(chunks) else 1.4)
         if best is None or cost < best[0]:
             best = cost, length
     size, items, run_items = best[1] * CHUNK, [], []

@@ -37,6 +37,54 @@ __device__ __forceinline__ float lin_decay(const LinStateDev& a, float z, int ch
   *one_minus = (1.0f - low) * ns;
   return logf(fmaxf(fmaf(1.0f - low, s, low), 1e-37f));
 }
+
+// The same in base 2 with the hardware's exponential and reciprocal, for the tensor-core form: bias and low are the
+// channel's.  Logarithms near 1 come from 2 artanh(u) = 2 (u + u^3 / 3 + ...), which keeps their relative error at
+// fp32's resolution (lg2.approx bounds the absolute error, and thousands of tokens would add that up).
+__device__ __forceinline__ float lin_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float lin_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float lin_lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+template <int MODE>
+__device__ __forceinline__ float lin_decay_log2(float y, float low, float inv_tau, float* one_minus) {
+  constexpr float LOG2E = 1.4426950408889634f;
+  const float e = lin_ex2(-fabsf(y) * LOG2E);
+  if constexpr (MODE == GATE_ROOT) {                       // -(max(-y, 0) log2 e + log2(1 + e)) / tau
+    const float u = e * lin_rcp(2.0f + e), u2 = u * u;
+    float p = fmaf(u2, 1.0f / 15, 1.0f / 13);
+    p = fmaf(u2, p, 1.0f / 11);
+    p = fmaf(u2, p, 1.0f / 9);
+    p = fmaf(u2, p, 1.0f / 7);
+    p = fmaf(u2, p, 1.0f / 5);
+    p = fmaf(u2, p, 1.0f / 3);
+    p = fmaf(u2 * u, p, u);
+    return fmaf(p, -2.0f * LOG2E, fminf(y, 0.0f) * LOG2E) * inv_tau;
+  } else {
+    // one reciprocal for 1 / (1 + e) and for u = k / (2 - k), k = room * num / (1 + e)
+    const float room = 1.0f - low, num = y >= 0.0f ? e : 1.0f, one = 1.0f + e, rn = room * num, den = fmaf(2.0f, one, -rn);
+    const float r = lin_rcp(one * den), inv = r * den, k = rn * inv, f = fmaf(room * inv, y >= 0.0f ? 1.0f : e, low);
+    *one_minus = k;
+    const float u = rn * one * r, u2 = u * u;               // k <= 1/4: u <= 1/7
+    float p = fmaf(u2, 1.0f / 9, 1.0f / 7);
+    p = fmaf(u2, p, 1.0f / 5);
+    p = fmaf(u2, p, 1.0f / 3);
+    p = fmaf(u2 * u, p, u);
+    return k <= 0.25f ? p * (-2.0f * LOG2E) : lin_lg2(fmaxf(f, 1e-37f));
+  }
+}
+__device__ __forceinline__ float lin_silu_fast(float x) { return x * lin_rcp(1.0f + lin_ex2(-1.4426950408889634f * x)); }
+
 __device__ __forceinline__ float lin_silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float lin_query(const LinStateDev& a, float q) { return (a.q_silu ? lin_silu(q) : q) * a.q_scale; }
 
