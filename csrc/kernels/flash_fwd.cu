@@ -438,6 +438,22 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       mbar_arrive_warp(p_ready(t));
     }
     // epilogue: O / l -> global, LSE
+    // The angles of 32 rows come in with coalesced loads, all on their way while the last product runs; they go through
+    // this warp's part of the P tile to the lanes: a row per lane and pair of columns, as the accumulator gives them.
+    const int pairs = p.o_cols >> 1, warp_row = q0 + t * C::BM + quad * 32;
+    const float2* turn = p.turn ? p.turn + ((long long)b * p.Tq + warp_row) * pairs : nullptr;
+    const bool turn_vec = turn && (pairs & 1) == 0 && (((uintptr_t)p.turn) & 15) == 0;
+    float4 angle[D / 32][8];
+    if (turn_vec) {
+#pragma unroll
+      for (int c = 0; c < D / 32; ++c)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int rr = i * 4 + (lane >> 3), at = c * 16 + (lane & 7) * 2;
+          angle[c][i] = make_float4(1.0f, 0.0f, 1.0f, 0.0f);
+          if (warp_row + rr < p.Tq && at < pairs) angle[c][i] = *reinterpret_cast<const float4*>(turn + (long long)rr * pairs + at);
+        }
+    }
     const bool have = my_hi > lo;
     if (have && ok) {
       if (!mbar_wait(o_done(t), (it - 1) & 1u, dead, p.status, 1320 + t)) ok = false;
@@ -447,8 +463,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const float inv_l = (l > 0.0f) ? 1.0f / l : 0.0f;
     const bool row_ok = qpos < p.Tq;
     __nv_bfloat16* orow = p.O + (long long)b * p.o_bs + (long long)qpos * p.o_ts + (long long)h * p.o_hs;
-    const float2* turn = p.turn && row_ok ? p.turn + ((long long)b * p.Tq + qpos) * (p.o_cols >> 1) : nullptr;
-#pragma unroll 1
+    uint8_t* stage = p_smem + quad * 4096;
+#pragma unroll
     for (int c = 0; c < D / 32; ++c) {
       uint32_t r[32];
       if (have && ok) {
@@ -459,12 +475,30 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
         for (int i = 0; i < 32; ++i) r[i] = 0u;
       }
+      if (turn_vec) {
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int rr = i * 4 + (lane >> 3), k = lane & 7;
+          *reinterpret_cast<float4*>(stage + rr * 128 + ((k ^ (rr & 7)) << 4)) = angle[c][i];
+        }
+        __syncwarp();
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          const float4 cs = *reinterpret_cast<const float4*>(stage + lane * 128 + ((k ^ (lane & 7)) << 4));
+          const float u0 = __uint_as_float(r[4 * k]), w0 = __uint_as_float(r[4 * k + 1]), u1 = __uint_as_float(r[4 * k + 2]), w1 = __uint_as_float(r[4 * k + 3]);
+          r[4 * k] = __float_as_uint(u0 * cs.x + w0 * cs.y);
+          r[4 * k + 1] = __float_as_uint(w0 * cs.x - u0 * cs.y);
+          r[4 * k + 2] = __float_as_uint(u1 * cs.z + w1 * cs.w);
+          r[4 * k + 3] = __float_as_uint(w1 * cs.z - u1 * cs.w);
+        }
+      }
       if (row_ok) {
-        if (turn) {
+        if (turn && !turn_vec) {
 #pragma unroll
           for (int i = 0; i < 16; ++i)
-            if (c * 16 + i < (p.o_cols >> 1)) {
-              const float2 cs = turn[c * 16 + i];
+            if (c * 16 + i < pairs) {
+              const float2 cs = turn[(long long)lane * pairs + c * 16 + i];
               const float u = __uint_as_float(r[2 * i]), w = __uint_as_float(r[2 * i + 1]);
               r[2 * i] = __float_as_uint(u * cs.x + w * cs.y);
               r[2 * i + 1] = __float_as_uint(w * cs.x - u * cs.y);

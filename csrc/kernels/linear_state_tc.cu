@@ -25,7 +25,7 @@ constexpr float LC_LIMIT = 100.0f;                        // largest exponent (b
 constexpr uint32_t T_K = 0, T_V = 32768, T_Q = 49152, T_A = 81920, T_S = 98304, T_END = 163840;
 constexpr uint32_t T_END_SUM = T_Q;                       // the summing pass has K and V only
 constexpr uint32_t T_SPLIT = 16384;                       // high part -> low part of Q and K
-constexpr uint32_t LC_MISC = (8 * 128 + 5 * 128 + 4 * LC) * 4 + 64;
+constexpr uint32_t LC_MISC = (8 * 128 + 5 * 128 + 4 * LC) * 4 + 64 + LC_THREADS * 8 * 12;      // and staged rows
 constexpr uint32_t TM_S = 0, TM_O = 128, TM_A = 256;      // TMEM columns
 
 struct ChunksDev {
@@ -114,50 +114,51 @@ linear_chunks_kernel(const ChunksDev c) {
 
   if (warp == 16) {
     // ------------------------------ issuer ------------------------------
-    if (lane == 0) {
-      const int ksteps = (D + 15) / 16;
-      const uint64_t dq = make_smem_desc_sw128(sb + T_Q, 16, 1024), dk = make_smem_desc_sw128(sb + T_K, 16, 1024);
-      const uint64_t da = make_smem_desc_sw128(sb + T_A, 16, 1024), ds = make_smem_desc_sw128(sb + T_S, 16384, 1024);
-      const uint64_t dv = make_smem_desc_sw128(sb + T_V, 8192, 1024), dkt = make_smem_desc_sw128(sb + T_K, 8192, 1024);
-      const uint32_t id_a = make_idesc_bf16(128, LC, 0, 0);   // rows 64 .. 127 of A and O are not used
-      const uint32_t id_o = make_idesc_bf16(128, 128, 0, 1), id_s = make_idesc_bf16(128, 128, 1, 1);
-      for (int n = 0; n < n_chunks; ++n) {
-        if (OUT) {
-          if (!mbar_wait(b_qk, n & 1, dead, c.status, 810)) break;
-          tc_fence_after();
-          if (*far_flag) {
-            mbar_arrive(bar_a);
-          } else {
-#pragma unroll 1
-            for (int p3 = 0; p3 < 3; ++p3) {
-              const uint64_t q = dq + (p3 == 2 ? T_SPLIT >> 4 : 0), k = dk + (p3 == 1 ? T_SPLIT >> 4 : 0);
-#pragma unroll
-              for (int kk = 0; kk < 8; ++kk)
-                if (kk < ksteps) umma_f16(tmem + TM_A, k_major(q, kk), k_major(k, kk), id_a, (p3 | kk) != 0);
-            }
-            umma_commit(bar_a);
-          }
-        }
-        if (!mbar_wait(b_sa, n & 1, dead, c.status, 811)) break;
+    const uint32_t mine = lane == 0;
+    const int ksteps = (D + 15) / 16;
+    const uint64_t dq = make_smem_desc_sw128(sb + T_Q, 16, 1024), dk = make_smem_desc_sw128(sb + T_K, 16, 1024);
+    const uint64_t da = make_smem_desc_sw128(sb + T_A, 16, 1024), ds = make_smem_desc_sw128(sb + T_S, 16384, 1024);
+    const uint64_t dv = make_smem_desc_sw128(sb + T_V, 8192, 1024), dkt = make_smem_desc_sw128(sb + T_K, 8192, 1024);
+    const uint32_t id_a = make_idesc_bf16(128, LC, 0, 0);   // rows 64 .. 127 of A and O are not used
+    const uint32_t id_o = make_idesc_bf16(128, 128, 0, 1), id_s = make_idesc_bf16(128, 128, 1, 1);
+    const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
+    for (int n = 0; n < n_chunks; ++n) {
+      if (OUT) {
+        if (!__all_sync(0xffffffffu, mbar_wait(b_qk, n & 1, dead, c.status, 810))) break;
         tc_fence_after();
-        if (OUT) {
-#pragma unroll 1
+        if (*far_flag) {
+          if (mine) mbar_arrive(bar_a);
+          __syncwarp();
+        } else {
+#pragma unroll
           for (int p3 = 0; p3 < 3; ++p3) {
-            const uint64_t q = dq + (p3 == 2 ? T_SPLIT >> 4 : 0), s = ds + (p3 == 1 ? 32768 >> 4 : 0);
+            const uint64_t q = dq + (p3 == 2 ? T_SPLIT >> 4 : 0), k = dk + (p3 == 1 ? T_SPLIT >> 4 : 0);
 #pragma unroll
             for (int kk = 0; kk < 8; ++kk)
-              if (kk < ksteps) umma_f16(tmem + TM_O, k_major(q, kk), mn_major(s, kk), id_o, (p3 | kk) != 0);
+              if (kk < ksteps) umma_f16_lane(mine, tm + TM_A, k_major(q, kk), k_major(k, kk), id_a, (p3 | kk) != 0);
           }
+          umma_commit_lane(mine, bar_a);
+        }
+      }
+      if (!__all_sync(0xffffffffu, mbar_wait(b_sa, n & 1, dead, c.status, 811))) break;
+      tc_fence_after();
+      if (OUT) {
 #pragma unroll
-          for (int kk = 0; kk < 2 * LC / 16; ++kk)
-            umma_f16(tmem + TM_O, da + (uint64_t)(((kk >> 2) * 8192 + (kk & 3) * 32) >> 4), mn_major(dv, kk & 3), id_o, 1);
-          umma_commit(bar_o);
+        for (int p3 = 0; p3 < 3; ++p3) {
+          const uint64_t q = dq + (p3 == 2 ? T_SPLIT >> 4 : 0), s = ds + (p3 == 1 ? 32768 >> 4 : 0);
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            if (kk < ksteps) umma_f16_lane(mine, tm + TM_O, k_major(q, kk), mn_major(s, kk), id_o, (p3 | kk) != 0);
         }
 #pragma unroll
         for (int kk = 0; kk < 2 * LC / 16; ++kk)
-          umma_f16(tmem + TM_S, mn_major(dkt + (kk >= 4 ? T_SPLIT >> 4 : 0), kk & 3), mn_major(dv, kk & 3), id_s, 1);
-        umma_commit(bar_s);
+          umma_f16_lane(mine, tm + TM_O, da + (uint64_t)(((kk >> 2) * 8192 + (kk & 3) * 32) >> 4), mn_major(dv, kk & 3), id_o, 1);
+        umma_commit_lane(mine, bar_o);
       }
+#pragma unroll
+      for (int kk = 0; kk < 2 * LC / 16; ++kk)
+        umma_f16_lane(mine, tm + TM_S, mn_major(dkt + (kk >= 4 ? T_SPLIT >> 4 : 0), kk & 3), mn_major(dv, kk & 3), id_s, 1);
+      umma_commit_lane(mine, bar_s);
     }
   } else {
     // ------------------------------ workers ------------------------------
@@ -191,51 +192,62 @@ linear_chunks_kernel(const ChunksDev c) {
     const float bias0 = mine ? a.bias[h * D + ch] : 0.0f, bias1 = mine ? a.bias[h * D + ch + 1] : 0.0f;
     const float low0 = MODE == GATE_BOUNDED && mine ? a.low[h * D + ch] : 0.0f, low1 = MODE == GATE_BOUNDED && mine ? a.low[h * D + ch + 1] : 0.0f;
 
-    auto fetch = [&](int n) {                             // a chunk's rows on their way to L2, 128 bytes per prefetch
+    // A chunk's rows: gates and one of keys and queries go to slots of this thread in shared memory, the others are
+    // asked for in L2 (128 bytes per prefetch).
+    constexpr bool STAGE_Q = OUT && MODE == GATE_BOUNDED;
+    const uint32_t st_z = smem_u32(bars) + 64 + tid * 8, st_w = smem_u32(bars) + 64 + 32768 + tid * 4;
+    const float2* sz = reinterpret_cast<const float2*>(bars + 16) + tid;
+    const uint32_t* sw = bars + 16 + 8192 + tid;
+    auto fetch = [&](int n) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int t = n * LC + tg * 8 + i;
+        if (mine && t < count) {
+          cp_async<8>(st_z + i * (LC_THREADS * 8), zp + (long long)t * a.ldz + ch);
+          if (STAGE_Q) cp_async<4>(st_w + i * (LC_THREADS * 4), qp + (long long)t * a.ldq + ch);
+          else if (MODE == GATE_ROOT) cp_async<4>(st_w + i * (LC_THREADS * 4), kp + (long long)t * a.ldk + ch);
+        }
+      }
       const int t = n * LC + (tid >> 3), i = tid & 7;
       if (t < count) {
-        if (i < 4) {
-          if (i * 32 < D) asm volatile("prefetch.global.L2 [%0];" ::"l"(zp + (long long)t * a.ldz + i * 32));
-          if (OUT && a.gate && i < 2 && i * 64 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(gp + (long long)t * a.ldg + i * 64));
-        } else if (i < 6) {
-          if ((i - 4) * 64 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(vp + (long long)t * a.ldv + (i - 4) * 64));
-          if (OUT && (i - 4) * 64 < D) asm volatile("prefetch.global.L2 [%0];" ::"l"(qp + (long long)t * a.ldq + (i - 4) * 64));
-        } else if (MODE == GATE_ROOT && (i - 6) * 64 < D) {
-          asm volatile("prefetch.global.L2 [%0];" ::"l"(kp + (long long)t * a.ldk + (i - 6) * 64));
+        if (i < 2) {
+          if (i * 64 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(vp + (long long)t * a.ldv + i * 64));
+        } else if (OUT && i < 4) {
+          if (a.gate && (i - 2) * 64 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(gp + (long long)t * a.ldg + (i - 2) * 64));
+        } else if (OUT && !STAGE_Q && i < 6) {
+          if ((i - 4) * 64 < D) asm volatile("prefetch.global.L2 [%0];" ::"l"(qp + (long long)t * a.ldq + (i - 4) * 64));
         }
       }
     };
     float b[8][2], kv[8][2], qv[8][2];
     auto gates = [&](int n) {                             // decays and their sums over eight tokens, keys, queries
-      float2 raw_z[8];
-      uint32_t raw_k[8], raw_q[8];
+      uint32_t raw_q[8];
+      if (OUT && !STAGE_Q) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int t = n * LC + tg * 8 + i;
-        raw_z[i] = make_float2(0.0f, 0.0f);
-        raw_k[i] = raw_q[i] = 0u;
-        if (mine && t < count) {
-          raw_z[i] = *reinterpret_cast<const float2*>(zp + (long long)t * a.ldz + ch);
-          if (MODE == GATE_ROOT) raw_k[i] = *reinterpret_cast<const uint32_t*>(kp + (long long)t * a.ldk + ch);
-          if (OUT) raw_q[i] = *reinterpret_cast<const uint32_t*>(qp + (long long)t * a.ldq + ch);
+        for (int i = 0; i < 8; ++i) {
+          const int t = n * LC + tg * 8 + i;
+          raw_q[i] = mine && t < count ? *reinterpret_cast<const uint32_t*>(qp + (long long)t * a.ldq + ch) : 0u;
         }
       }
+      cp_async_wait_all();
       float sum0 = 0.0f, sum1 = 0.0f;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const bool in = mine && n * LC + tg * 8 + i < count;
+        const bool in = mine && n * LC + tg * 8 + i < count;      // otherwise the slot holds an earlier chunk's row
+        const float2 z = in ? sz[i * LC_THREADS] : make_float2(0.0f, 0.0f);
+        const uint32_t w = in && (STAGE_Q || MODE == GATE_ROOT) ? sw[i * LC_THREADS] : 0u;
         float k0 = 0.0f, k1 = 0.0f;
-        const float g0 = lin_decay_log2<MODE>(raw_z[i].x + bias0, low0, a.inv_tau, &k0);
-        const float g1 = lin_decay_log2<MODE>(raw_z[i].y + bias1, low1, a.inv_tau, &k1);
+        const float g0 = lin_decay_log2<MODE>(z.x + bias0, low0, a.inv_tau, &k0);
+        const float g1 = lin_decay_log2<MODE>(z.y + bias1, low1, a.inv_tau, &k1);
         if (MODE == GATE_ROOT) {
-          const float2 k = unpack_bf16x2(raw_k[i]);
+          const float2 k = unpack_bf16x2(w);
           k0 = k.x;
           k1 = k.y;
         }
         kv[i][0] = in ? k0 : 0.0f;
         kv[i][1] = in ? k1 : 0.0f;
         if (OUT) {
-          const float2 q = unpack_bf16x2(raw_q[i]);
+          const float2 q = unpack_bf16x2(STAGE_Q ? w : raw_q[i]);
           qv[i][0] = (a.q_silu ? lin_silu_fast(q.x) : q.x) * a.q_scale;
           qv[i][1] = (a.q_silu ? lin_silu_fast(q.y) : q.y) * a.q_scale;
         }
