@@ -123,7 +123,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "cgk_kv_gather": [vp, i, i, i, i, vp, vp, vp],
         "cgk_kv_rows_attention": [vp, vp, ll, i, vp, ll, vp, i, i, f, i, i, i, vp, vp],
         "cgk_linear_state": [vp, i, vp],
-        "cgk_linear_chunks": [vp, vp, i, vp, i, vp, vp],
+        "cgk_linear_chunks": [vp, i, vp, i, vp, i, vp, vp],
         "cgk_linear_chunks_ok": [i, i],
         "cgk_stream_norms": [vp, vp],
         "cgk_softcap": [vp, ll, f, vp],

@@ -136,18 +136,18 @@ def _chunked(rule: StateRule, x: Operands) -> bool:
     return all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (x.q, x.k, x.v, x.gate, x.z))
 
 
-def _advance_chunks(a: LinearStateArgs, rule: StateRule, batch, device):
+def _advance_chunks(a: LinearStateArgs, rule: StateRule, batch, rows: int, device):
     key = ("stretches", rule.heads)
     if key not in batch.memo:
-        rows = [g.start + i * g.count for g in batch.prompts for i in range(g.sequences)]
-        items, run_items, cut = stretches([g.count for g in batch.prompts for _ in range(g.sequences)], rule.heads, rows)
+        first = [g.start + i * g.count for g in batch.prompts for i in range(g.sequences)]
+        items, run_items, cut = stretches([g.count for g in batch.prompts for _ in range(g.sequences)], rule.heads, first)
         flat = torch.tensor([v for t in items + run_items for v in t], dtype=torch.int32).to(device)
         batch.memo[key] = flat, len(items), len(run_items), cut
     flat, n, runs, cut = batch.memo[key]
     L, scratch = _lib.lib(), None
     if cut:
         scratch = torch.empty(L.cgk_linear_chunks_scratch_floats(n, rule.heads, rule.dim, rule.vdim), dtype=torch.float32, device=device)
-    _lib.check(L.cgk_linear_chunks(ctypes.byref(a), flat.data_ptr(), n, flat[4 * n:].data_ptr(), runs, _lib.ptr(scratch), _lib.stream_ptr()),
+    _lib.check(L.cgk_linear_chunks(ctypes.byref(a), rows, flat.data_ptr(), n, flat[4 * n:].data_ptr(), runs, _lib.ptr(scratch), _lib.stream_ptr()),
                "cgk_linear_chunks")
     _lib.count_launch(3 if cut else 1)
 
@@ -161,7 +161,7 @@ def advance(rule: StateRule, x: Operands, state, batch, out):
     if not x.q.is_cuda:
         return _advance_cpu(rule, x, state, slot, pos, runs, out)
     if batch.prompts and _chunked(rule, x) and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0:
-        _advance_chunks(_args(rule, x, state, slot, pos, None, out), rule, batch, out.device)
+        _advance_chunks(_args(rule, x, state, slot, pos, None, out), rule, batch, x.q.shape[0], out.device)
         runs = runs[sum(g.sequences for g in batch.prompts):]
     n = x.q.shape[0] if runs is None else runs.shape[0]
     if n:

@@ -2,11 +2,13 @@
 //
 // With b_t the logarithm of the decay since the start of a chunk (per state row), r its value in the chunk's middle,
 //     Q = q 2^(b - r),  K = k 2^(r - b),  A = tril(Q K^T),  O = A V + Q (2^r S),  S' = 2^(b_end - r) (2^r S + K^T V)
-// so a chunk takes four products.  The state stays in TMEM in fp32 from chunk to chunk (times a factor per row that is kept
-// beside it); every fp32 operand enters the tensor core as the sum of two bf16 numbers (three products for two such
-// operands, the smallest one is dropped), so the sums see 16 bits of each factor.  Where a decay is so strong that
-// the exponents could leave fp32's range, A is formed term by term with b_t - b_s <= 0, and Q and K take the
-// chunk's ends as their references.
+// so a chunk takes four products.  The state stays in TMEM in fp32 from chunk to chunk (transposed: lanes are the elements
+// of v; times a factor per state row that is kept beside it).  Every fp32 operand enters the tensor core as the sum of
+// two bf16 numbers, so the sums see 16 bits of each factor; the two parts of Q, K and A are stacked in one tile, which
+// makes the partial products one wider instruction:
+//     [Qh; Ql] [Kh; Kl]^T  -> A in four quarters        Sh [Qh; Ql]^T, Sl Qh^T, V^T [Ah; Al]^T  -> O^T in two halves
+// Where a decay is so strong that the exponents could leave fp32's range, A is formed term by term with
+// b_t - b_s <= 0, and Q and K take the chunk's ends as their references.
 //
 // One CTA walks the chunks of one (stretch of a run, head).  A long run is cut into stretches that run side by side: a
 // first pass sums up what each stretch adds to the state, a second one turns that into the stretches' first states.
@@ -19,14 +21,14 @@
 namespace cgk {
 namespace {
 
-constexpr int LC = 64, LC_THREADS = 512;
+constexpr int LC = 64, LC_THREADS = 512;                  // tokens of a chunk; worker threads
 constexpr float LC_LIMIT = 100.0f;                        // largest exponent (base 2) of a factor
-// shared memory: operand tiles of 128-byte rows in blocks of 64 columns (bytes)
-constexpr uint32_t T_K = 0, T_V = 32768, T_Q = 49152, T_A = 81920, T_S = 98304, T_END = 163840;
-constexpr uint32_t T_END_SUM = T_Q;                       // the summing pass has K and V only
-constexpr uint32_t T_SPLIT = 16384;                       // high part -> low part of Q and K
-constexpr uint32_t LC_MISC = (8 * 128 + 5 * 128 + 4 * LC) * 4 + 64 + LC_THREADS * 8 * 12;      // and staged rows
-constexpr uint32_t TM_S = 0, TM_O = 128, TM_A = 256;      // TMEM columns
+// shared memory (bytes): operand tiles of 128-byte rows in blocks of 64 columns, then rows as they come from memory
+constexpr uint32_t T_Q = 0, T_K = 32768, T_V = 65536, T_A = 81920, T_A2 = 98304, R_Z = 106496, R_W = R_Z + 32768, R_X = R_W + 16384, LC_MISC = R_X + 16384;
+constexpr uint32_t LC_SMEM = LC_MISC + (8 * 128 + 5 * 128 + 4 * LC) * 4 + 128 + 1024;
+constexpr uint32_t T_SPLIT = 8192;                        // high part -> low part of Q, K and A: 64 rows further
+// TMEM columns: state, its two parts, O in two halves, A in four quarters
+constexpr uint32_t TM_S = 0, TM_SH = 128, TM_SL = 192, TM_O = 256, TM_A = 384;
 
 struct ChunksDev {
   LinStateDev a;
@@ -47,7 +49,7 @@ __device__ __forceinline__ uint32_t pair_at(int row, int col, int rows) {
 }
 
 // operand descriptors of consecutive 16-wide steps differ by constants in the address field
-__device__ __forceinline__ uint64_t k_major(uint64_t d, int kk) { return d + (uint64_t)(((kk >> 2) * (LC * 128) + (kk & 3) * 32) >> 4); }
+__device__ __forceinline__ uint64_t k_major(uint64_t d, int kk) { return d + (uint64_t)(((kk >> 2) * 16384 + (kk & 3) * 32) >> 4); }
 __device__ __forceinline__ uint64_t mn_major(uint64_t d, int kk) { return d + (uint64_t)((kk * 2048) >> 4); }
 
 // meeting point of the sixteen worker warps, plain and with a vote
@@ -63,33 +65,44 @@ __device__ __forceinline__ bool lc_any(bool v) {
   return r != 0;
 }
 
-// Warps 0 .. 15 prepare operands and read results, warp 16 issues the products.
+// 16 values per lane -> their sums over the warp: lane l gets the sum of value (l >> 1).
+__device__ __forceinline__ float sum_over_lanes(float (&v)[16], int lane) {
+#pragma unroll
+  for (int half = 8; half >= 1; half >>= 1) {
+    const bool upper = (lane & (2 * half)) != 0;
+#pragma unroll
+    for (int i = 0; i < half; ++i) {
+      const float send = upper ? v[i] : v[i + half];
+      v[i] = (upper ? v[i + half] : v[i]) + __shfl_xor_sync(0xffffffffu, send, 2 * half);
+    }
+  }
+  return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+}
+
+// Warps 0 .. 15 prepare operands and read results, warp 16 issues the products, warp 17 brings gates, queries and keys.
 template <bool OUT, int MODE>
-__global__ void __launch_bounds__(LC_THREADS + 32, 1)
-linear_chunks_kernel(const ChunksDev c) {
+__global__ void __launch_bounds__(LC_THREADS + 128, 1)
+linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
+                     const __grid_constant__ CUtensorMap tm_v, const ChunksDev c) {
   const LinStateDev& a = c.a;
   extern __shared__ uint8_t lc_raw[];
   uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lc_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sb = smem_u32(sm);
-  constexpr uint32_t END = OUT ? T_END : T_END_SUM;
-  float* part = reinterpret_cast<float*>(sm + END);       // [8][128] decay of eight tokens
-  float* rq = part + 8 * 128;                             // [128] references of Q and K
-  float* rk = rq + 128;
-  float* pend = rk + 128;                                 // [2][128] factor of the state in TMEM, by parity of the chunk
-  float* tot = pend + 256;                                // [128] decay of all chunks
-  float* red = tot + 128;                                 // [4][64]
+  float* part = reinterpret_cast<float*>(sm + LC_MISC);   // [8][128] decay of eight tokens
+  float* f0 = part + 8 * 128;                             // [128] factors of the state: pending, of K's reference
+  float* fk = f0 + 128;
+  float* red = fk + 128;                                  // [4][64]
   uint32_t* bars = reinterpret_cast<uint32_t*>(red + 4 * LC);
-  const uint32_t b_qk = smem_u32(bars), b_sa = b_qk + 8, bar_a = b_qk + 16, bar_o = b_qk + 24, bar_s = b_qk + 32;
-  volatile uint32_t* tmem_slot = bars + 10;
-  volatile int* dead = reinterpret_cast<volatile int*>(bars + 11);
-  volatile int* far_flag = reinterpret_cast<volatile int*>(bars + 12);
+  const uint32_t b_qk = smem_u32(bars), b_sa = b_qk + 8, bar_a = b_qk + 16, bar_o = b_qk + 24, bar_s = b_qk + 32, b_raw = b_qk + 40, b_free = b_qk + 48, b_v = b_qk + 56;
+  volatile uint32_t* tmem_slot = bars + 16;
+  volatile int* dead = reinterpret_cast<volatile int*>(bars + 17);
+  volatile int* far_flag = reinterpret_cast<volatile int*>(bars + 18);
 
   const int* item = c.items + 4 * blockIdx.y;
   const int row0 = item[0], count = item[1], last = item[3], h = blockIdx.x;
   if (!OUT && last) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int D = a.D, V = a.V, n_chunks = (count + LC - 1) / LC;
-  constexpr uint32_t COLS = OUT ? 512 : 128;
 
   if (tid == 0) {
     mbar_init(b_qk, 16);
@@ -97,30 +110,49 @@ linear_chunks_kernel(const ChunksDev c) {
     mbar_init(bar_a, 1);
     mbar_init(bar_o, 1);
     mbar_init(bar_s, 1);
+    mbar_init(b_raw, 1);
+    mbar_init(b_free, 16);
+    mbar_init(b_v, 1);
     *dead = 0;
     mbar_fence_init();
   }
   if (warp == 0) {
-    tmem_alloc(smem_u32((const void*)tmem_slot), COLS);
+    tmem_alloc(smem_u32((const void*)tmem_slot), 512);
     tmem_relinquish();
   }
-  if (V < 128 && tid < LC_THREADS)                        // columns that are not loaded
-    for (uint32_t i = tid; i < 1024; i += LC_THREADS) reinterpret_cast<uint4*>(sm + T_V)[i] = make_uint4(0, 0, 0, 0);
-  if (tid < 128) { pend[tid] = 0.0f; tot[tid] = 0.0f; }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
-
-  if (warp == 16) {
+  // 640 threads are launched with 96 registers each; the last warpgroup leaves some of its share to the workers
+  if (warp >= 16) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 56;");
+   if (warp == 17) {
+    // ------------------------------ loader ------------------------------
+    // 64 rows at a time; what lies behind the end of the run is another run's (or zero) and is not used
+    if (lane == 0) {
+      const int v_blocks = (V + 63) / 64;
+      for (int n = 0; n < n_chunks; ++n) {
+        const int row = row0 + n * LC;
+        if (n > 0 && !mbar_wait(b_free, (n - 1) & 1, dead, c.status, 820)) break;
+        mbar_expect_tx(b_raw, LC * D * (4 + (OUT ? 2 : 0) + (MODE == GATE_ROOT ? 2 : 0)));
+        tma_load_2d(sb + R_Z, &tm_z, b_raw, h * D, row);
+        if (OUT) tma_load_2d(sb + R_W, &tm_q, b_raw, h * D, row);
+        if (MODE == GATE_ROOT) tma_load_2d(sb + R_X, &tm_k, b_raw, h * D, row);
+        if (n > 0 && !mbar_wait(bar_s, (n - 1) & 1, dead, c.status, 822)) break;
+        mbar_expect_tx(b_v, v_blocks * 8192);
+        for (int i = 0; i < v_blocks; ++i) tma_load_2d(sb + T_V + i * 8192, &tm_v, b_v, h * V + i * 64, row);
+      }
+    }
+  } else if (warp == 16) {
     // ------------------------------ issuer ------------------------------
     const uint32_t mine = lane == 0;
     const int ksteps = (D + 15) / 16;
     const uint64_t dq = make_smem_desc_sw128(sb + T_Q, 16, 1024), dk = make_smem_desc_sw128(sb + T_K, 16, 1024);
-    const uint64_t da = make_smem_desc_sw128(sb + T_A, 16, 1024), ds = make_smem_desc_sw128(sb + T_S, 16384, 1024);
-    const uint64_t dv = make_smem_desc_sw128(sb + T_V, 8192, 1024), dkt = make_smem_desc_sw128(sb + T_K, 8192, 1024);
-    const uint32_t id_a = make_idesc_bf16(128, LC, 0, 0);   // rows 64 .. 127 of A and O are not used
-    const uint32_t id_o = make_idesc_bf16(128, 128, 0, 1), id_s = make_idesc_bf16(128, 128, 1, 1);
+    const uint64_t da = make_smem_desc_sw128(sb + T_A, 16, 1024), da2 = make_smem_desc_sw128(sb + T_A2, 16, 1024);
+    const uint64_t dv = make_smem_desc_sw128(sb + T_V, 8192, 1024), dkt = make_smem_desc_sw128(sb + T_K, 16384, 1024);
+    const uint32_t id_kk = make_idesc_bf16(128, 128, 0, 0), id_kk64 = make_idesc_bf16(128, 64, 0, 0);
+    const uint32_t id_mk = make_idesc_bf16(128, 128, 1, 0), id_mk64 = make_idesc_bf16(128, 64, 1, 0), id_mm = make_idesc_bf16(128, 128, 1, 1);
     const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
     for (int n = 0; n < n_chunks; ++n) {
       if (OUT) {
@@ -131,148 +163,96 @@ linear_chunks_kernel(const ChunksDev c) {
           __syncwarp();
         } else {
 #pragma unroll
-          for (int p3 = 0; p3 < 3; ++p3) {
-            const uint64_t q = dq + (p3 == 2 ? T_SPLIT >> 4 : 0), k = dk + (p3 == 1 ? T_SPLIT >> 4 : 0);
-#pragma unroll
-            for (int kk = 0; kk < 8; ++kk)
-              if (kk < ksteps) umma_f16_lane(mine, tm + TM_A, k_major(q, kk), k_major(k, kk), id_a, (p3 | kk) != 0);
-          }
+          for (int kk = 0; kk < 8; ++kk)
+            if (kk < ksteps) umma_f16_lane(mine, tm + TM_A, k_major(dq, kk), k_major(dk, kk), id_kk, kk != 0);
           umma_commit_lane(mine, bar_a);
         }
       }
-      if (!__all_sync(0xffffffffu, mbar_wait(b_sa, n & 1, dead, c.status, 811))) break;
+      if (!__all_sync(0xffffffffu, mbar_wait(b_v, n & 1, dead, c.status, 812) && mbar_wait(b_sa, n & 1, dead, c.status, 811))) break;
       tc_fence_after();
       if (OUT) {
 #pragma unroll
-        for (int p3 = 0; p3 < 3; ++p3) {
-          const uint64_t q = dq + (p3 == 2 ? T_SPLIT >> 4 : 0), s = ds + (p3 == 1 ? 32768 >> 4 : 0);
+        for (int kk = 0; kk < 8; ++kk)
+          if (kk < ksteps) umma_f16_ts_lane(mine, tm + TM_O, tm + TM_SH + kk * 8, k_major(dq, kk), id_kk, kk != 0);
 #pragma unroll
-          for (int kk = 0; kk < 8; ++kk)
-            if (kk < ksteps) umma_f16_lane(mine, tm + TM_O, k_major(q, kk), mn_major(s, kk), id_o, (p3 | kk) != 0);
-        }
+        for (int kk = 0; kk < 8; ++kk)
+          if (kk < ksteps) umma_f16_ts_lane(mine, tm + TM_O, tm + TM_SL + kk * 8, k_major(dq, kk), id_kk64, 1);
 #pragma unroll
-        for (int kk = 0; kk < 2 * LC / 16; ++kk)
-          umma_f16_lane(mine, tm + TM_O, da + (uint64_t)(((kk >> 2) * 8192 + (kk & 3) * 32) >> 4), mn_major(dv, kk & 3), id_o, 1);
+        for (int kk = 0; kk < LC / 16; ++kk) umma_f16_lane(mine, tm + TM_O, mn_major(dv, kk), da + kk * 2, id_mk, 1);
+#pragma unroll
+        for (int kk = 0; kk < LC / 16; ++kk) umma_f16_lane(mine, tm + TM_O, mn_major(dv, kk), da2 + kk * 2, id_mk64, 1);
         umma_commit_lane(mine, bar_o);
       }
 #pragma unroll
       for (int kk = 0; kk < 2 * LC / 16; ++kk)
-        umma_f16_lane(mine, tm + TM_S, mn_major(dkt + (kk >= 4 ? T_SPLIT >> 4 : 0), kk & 3), mn_major(dv, kk & 3), id_s, 1);
+        umma_f16_lane(mine, tm + TM_S, mn_major(dv, kk & 3), mn_major(dkt + (kk >= 4 ? T_SPLIT >> 4 : 0), kk & 3), id_mm, 1);
       umma_commit_lane(mine, bar_s);
     }
+   }
   } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 104;");
     // ------------------------------ workers ------------------------------
-    const int quad = warp & 3, cg = warp >> 2, srow = quad * 32 + lane;
+    const int quad = warp & 3, cg = warp >> 2, lrow = quad * 32 + lane;       // TMEM lane: an element of v, or a row of A
     const uint32_t lanes = (uint32_t)(quad * 32) << 16;
     const int p0 = a.pos[row0];
     const long long slot = CGK_IDX(a.slot[row0], a.slots);
     {
-      // first state -> TMEM: lane = state row, this warp's 32 columns
+      // first state -> TMEM: this warp's 32 state rows
       const float* src = nullptr;
       if (OUT && c.start) src = c.start + ((long long)blockIdx.y * a.heads + h) * D * V;
       else if (OUT && p0 > 0) src = a.state + ((slot * a.history + p0 % a.history) * a.heads + h) * (long long)D * V;
       uint32_t r[32];
 #pragma unroll
-      for (int j = 0; j < 32; j += 4) {
-        float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        if (src && srow < D && cg * 32 + j < V) ldv<4>(src + (long long)srow * V + cg * 32 + j, v);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) r[j + e] = __float_as_uint(v[e]);
-      }
+      for (int j = 0; j < 32; ++j)
+        r[j] = src && lrow < V && cg * 32 + j < D ? __float_as_uint(src[(long long)(cg * 32 + j) * V + lrow]) : 0u;
       tmem_st32(tmem + TM_S + lanes + cg * 32, r);
       tmem_st_wait();
     }
-    const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(a.q) + (long long)row0 * a.ldq + h * D;
-    const __nv_bfloat16* kp = reinterpret_cast<const __nv_bfloat16*>(a.k) + (MODE == GATE_ROOT ? (long long)row0 * a.ldk + h * D : 0);
-    const __nv_bfloat16* vp = reinterpret_cast<const __nv_bfloat16*>(a.v) + (long long)row0 * a.ldv + h * V;
-    const __nv_bfloat16* gp = reinterpret_cast<const __nv_bfloat16*>(a.gate) + (a.gate ? (long long)row0 * a.ldg + h * V : 0);
-    const float* zp = a.z + (long long)row0 * a.ldz + h * D;
+    // results leave with two 16-byte pieces per thread: rows cg * 16 + (0, 8) + .., columns o_col ..
+    const int o_row = cg * 16 + (quad * 32 + lane) / 16, o_col = (lane & 15) * 8;
+    const bool o_mine = o_col < V;
+    const __nv_bfloat16* gp = reinterpret_cast<const __nv_bfloat16*>(a.gate) + (a.gate ? (long long)row0 * a.ldg + h * V + o_col : 0);
+    __nv_bfloat16* op = reinterpret_cast<__nv_bfloat16*>(a.out) + (long long)row0 * a.ldo + h * V + o_col;
     const int ch = (tid & 63) * 2, tg = tid >> 6;         // two state rows, eight tokens
     const bool mine = ch < D;
     const float bias0 = mine ? a.bias[h * D + ch] : 0.0f, bias1 = mine ? a.bias[h * D + ch + 1] : 0.0f;
     const float low0 = MODE == GATE_BOUNDED && mine ? a.low[h * D + ch] : 0.0f, low1 = MODE == GATE_BOUNDED && mine ? a.low[h * D + ch + 1] : 0.0f;
+    bool ok = true;                                       // after a wait that ran out a warp still comes to every meeting point
 
-    // A chunk's rows: gates and one of keys and queries go to slots of this thread in shared memory, the others are
-    // asked for in L2 (128 bytes per prefetch).
-    constexpr bool STAGE_Q = OUT && MODE == GATE_BOUNDED;
-    const uint32_t st_z = smem_u32(bars) + 64 + tid * 8, st_w = smem_u32(bars) + 64 + 32768 + tid * 4;
-    const float2* sz = reinterpret_cast<const float2*>(bars + 16) + tid;
-    const uint32_t* sw = bars + 16 + 8192 + tid;
-    auto fetch = [&](int n) {
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int t = n * LC + tg * 8 + i;
-        if (mine && t < count) {
-          cp_async<8>(st_z + i * (LC_THREADS * 8), zp + (long long)t * a.ldz + ch);
-          if (STAGE_Q) cp_async<4>(st_w + i * (LC_THREADS * 4), qp + (long long)t * a.ldq + ch);
-          else if (MODE == GATE_ROOT) cp_async<4>(st_w + i * (LC_THREADS * 4), kp + (long long)t * a.ldk + ch);
-        }
-      }
-      const int t = n * LC + (tid >> 3), i = tid & 7;
-      if (t < count) {
-        if (i < 2) {
-          if (i * 64 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(vp + (long long)t * a.ldv + i * 64));
-        } else if (OUT && i < 4) {
-          if (a.gate && (i - 2) * 64 < V) asm volatile("prefetch.global.L2 [%0];" ::"l"(gp + (long long)t * a.ldg + (i - 2) * 64));
-        } else if (OUT && !STAGE_Q && i < 6) {
-          if ((i - 4) * 64 < D) asm volatile("prefetch.global.L2 [%0];" ::"l"(qp + (long long)t * a.ldq + (i - 4) * 64));
-        }
-      }
-    };
-    float b[8][2], kv[8][2], qv[8][2];
+    float kv[8][2], qv[8][2], pend[2] = {0.0f, 0.0f}, tot[2] = {0.0f, 0.0f};
     auto gates = [&](int n) {                             // decays and their sums over eight tokens, keys, queries
-      uint32_t raw_q[8];
-      if (OUT && !STAGE_Q) {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const int t = n * LC + tg * 8 + i;
-          raw_q[i] = mine && t < count ? *reinterpret_cast<const uint32_t*>(qp + (long long)t * a.ldq + ch) : 0u;
-        }
-      }
-      cp_async_wait_all();
+      ok &= mbar_wait(b_raw, n & 1, dead, c.status, 821);
       float sum0 = 0.0f, sum1 = 0.0f;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const bool in = mine && n * LC + tg * 8 + i < count;      // otherwise the slot holds an earlier chunk's row
-        const float2 z = in ? sz[i * LC_THREADS] : make_float2(0.0f, 0.0f);
-        const uint32_t w = in && (STAGE_Q || MODE == GATE_ROOT) ? sw[i * LC_THREADS] : 0u;
+        const int t = tg * 8 + i;
+        const bool in = mine && n * LC + t < count;       // otherwise the place holds an earlier chunk's row
+        const float2 z = in ? *reinterpret_cast<const float2*>(sm + R_Z + (t * D + ch) * 4) : make_float2(0.0f, 0.0f);
         float k0 = 0.0f, k1 = 0.0f;
         const float g0 = lin_decay_log2<MODE>(z.x + bias0, low0, a.inv_tau, &k0);
         const float g1 = lin_decay_log2<MODE>(z.y + bias1, low1, a.inv_tau, &k1);
         if (MODE == GATE_ROOT) {
-          const float2 k = unpack_bf16x2(w);
+          const float2 k = unpack_bf16x2(in ? *reinterpret_cast<const uint32_t*>(sm + R_X + (t * D + ch) * 2) : 0u);
           k0 = k.x;
           k1 = k.y;
         }
         kv[i][0] = in ? k0 : 0.0f;
         kv[i][1] = in ? k1 : 0.0f;
         if (OUT) {
-          const float2 q = unpack_bf16x2(STAGE_Q ? w : raw_q[i]);
+          const float2 q = unpack_bf16x2(in ? *reinterpret_cast<const uint32_t*>(sm + R_W + (t * D + ch) * 2) : 0u);
           qv[i][0] = (a.q_silu ? lin_silu_fast(q.x) : q.x) * a.q_scale;
           qv[i][1] = (a.q_silu ? lin_silu_fast(q.y) : q.y) * a.q_scale;
         }
         sum0 += in ? g0 : 0.0f;
         sum1 += in ? g1 : 0.0f;
-        b[i][0] = sum0;
-        b[i][1] = sum1;
+        if (mine) *reinterpret_cast<float2*>(sm + R_Z + (t * D + ch) * 4) = make_float2(sum0, sum1);      // read back by this thread
       }
       *reinterpret_cast<float2*>(part + tg * 128 + ch) = make_float2(sum0, sum1);
     };
-    fetch(0);
     gates(0);
-    bool ok = true;                                       // after a wait that ran out a warp still comes to every meeting point
 
     for (int n = 0; n < n_chunks; ++n) {
       const int t0 = n * LC, left = min(LC, count - t0);
-      // values: two 16-byte pieces per thread
-      uint4 vv[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int j = tid + i * LC_THREADS, t = j >> 4, col = (j & 15) * 8;
-        vv[i] = make_uint4(0, 0, 0, 0);
-        if (t < left && col < V) vv[i] = *reinterpret_cast<const uint4*>(vp + (long long)(t0 + t) * a.ldv + col);
-      }
-      if (n + 1 < n_chunks) fetch(n + 1);
       // the previous chunk's products are done with the tiles and the state
       if (n > 0) ok &= mbar_wait(bar_s, (n - 1) & 1, dead, c.status, 802);
       tc_fence_after();
@@ -286,196 +266,211 @@ linear_chunks_kernel(const ChunksDev c) {
         end[1] += s.y;
         if (g == 3) { mid[0] = end[0]; mid[1] = end[1]; }
       }
-#pragma unroll
-      for (int i = 0; i < 8; ++i) { b[i][0] += before[0]; b[i][1] += before[1]; }
+      auto sum_at = [&](int i) {                          // decay up to and with this thread's token i
+        const float2 s = mine ? *reinterpret_cast<const float2*>(sm + R_Z + ((tg * 8 + i) * D + ch) * 4) : make_float2(0.0f, 0.0f);
+        return make_float2(s.x + before[0], s.y + before[1]);
+      };
       bool far = false;
       if (OUT) far = lc_any(fmaxf(-mid[0], -mid[1]) > LC_LIMIT || fmaxf(mid[0] - end[0], mid[1] - end[1]) > LC_LIMIT);
       if (far) {
-        // A term by term, into its tile at once: row tid / 8, columns 8 (tid % 8) ..
-        float* fb = reinterpret_cast<float*>(sm + T_S);
-        float* fq = fb + LC * 128;
-        float* fk = reinterpret_cast<float*>(sm + T_K);
+        // A term by term: row tid / 8, columns 8 (tid % 8) ..; scratch space: the tiles of Q and K, and b in its own rows
+        float* fx = reinterpret_cast<float*>(sm + T_Q);
+        float* fy = reinterpret_cast<float*>(sm + T_K);
+        float* fb = reinterpret_cast<float*>(sm + R_Z);
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const int at = (tg * 8 + i) * 128 + ch;
-          *reinterpret_cast<float2*>(fb + at) = make_float2(b[i][0], b[i][1]);
-          *reinterpret_cast<float2*>(fq + at) = make_float2(qv[i][0], qv[i][1]);
-          *reinterpret_cast<float2*>(fk + at) = make_float2(kv[i][0], kv[i][1]);
+          *reinterpret_cast<float2*>(fx + at) = make_float2(qv[i][0], qv[i][1]);
+          *reinterpret_cast<float2*>(fy + at) = make_float2(kv[i][0], kv[i][1]);
+          if (mine) *reinterpret_cast<float2*>(fb + (tg * 8 + i) * D + ch) = sum_at(i);
         }
+        before[0] = before[1] = 0.0f;                     // b's rows are complete now
         lc_meet();
         const int t = tid >> 3, s0 = (tid & 7) * 8;
-#pragma unroll 1
+        uint32_t hi[4], lo[4];
+#pragma unroll
         for (int j = 0; j < 4; ++j) {
           float x[2] = {0.0f, 0.0f};
 #pragma unroll
-          for (int e2 = 0; e2 < 2; ++e2) {
-            const int s = s0 + 2 * j + e2;
+          for (int i = 0; i < 2; ++i) {
+            const int s = s0 + 2 * j + i;
             if (s <= t)
-              for (int e = 0; e < D; ++e) x[e2] = fmaf(fq[t * 128 + e] * fk[s * 128 + e], exp2f(fb[t * 128 + e] - fb[s * 128 + e]), x[e2]);
+#pragma unroll 1
+              for (int e = 0; e < D; ++e) x[i] = fmaf(fx[t * 128 + e] * fy[s * 128 + e], exp2f(fb[t * D + e] - fb[s * D + e]), x[i]);
           }
-          uint32_t hh, ll;
-          split2(x[0], x[1], hh, ll);
-          *reinterpret_cast<uint32_t*>(sm + T_A + pair_at(t, s0 + 2 * j, LC)) = hh;
-          *reinterpret_cast<uint32_t*>(sm + T_A + 8192 + pair_at(t, s0 + 2 * j, LC)) = ll;
+          split2(x[0], x[1], hi[j], lo[j]);
         }
         lc_meet();
+        const uint32_t at = sw128_offset(t, s0 >> 3);
+        *reinterpret_cast<uint4*>(sm + T_A + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(sm + T_A + T_SPLIT + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        *reinterpret_cast<uint4*>(sm + T_A2 + at) = make_uint4(0, 0, 0, 0);
       }
       const float ref_q[2] = {far ? 0.0f : mid[0], far ? 0.0f : mid[1]};
       const float ref_k[2] = {far || !OUT ? end[0] : mid[0], far || !OUT ? end[1] : mid[1]};
       if (tg == 0) {
-        rq[ch] = ref_q[0]; rq[ch + 1] = ref_q[1];
-        rk[ch] = ref_k[0]; rk[ch + 1] = ref_k[1];
-        float* next = pend + ((n + 1) & 1) * 128 + ch;
-        next[0] = end[0] - ref_k[0];
-        next[1] = end[1] - ref_k[1];
-        tot[ch] += end[0];
-        tot[ch + 1] += end[1];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          f0[ch + i] = exp2f(pend[i]);
+          fk[ch + i] = exp2f(ref_k[i]);                   // Q's reference is the same, or 0
+        }
         if (tid == 0) *far_flag = far;
       }
 #pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        pend[i] = end[i] - ref_k[i];
+        tot[i] += end[i];
+      }
+#pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const uint32_t at = pair_at(tg * 8 + i, ch, LC);
+        const uint32_t at = pair_at(tg * 8 + i, ch, 128);
+        const float2 b = sum_at(i);
         uint32_t hi, lo;
-        split2(kv[i][0] * fast_exp2(ref_k[0] - b[i][0]), kv[i][1] * fast_exp2(ref_k[1] - b[i][1]), hi, lo);
+        split2(kv[i][0] * fast_exp2(ref_k[0] - b.x), kv[i][1] * fast_exp2(ref_k[1] - b.y), hi, lo);
         *reinterpret_cast<uint32_t*>(sm + T_K + at) = hi;
         *reinterpret_cast<uint32_t*>(sm + T_K + T_SPLIT + at) = lo;
         if (OUT) {
-          split2(qv[i][0] * fast_exp2(b[i][0] - ref_q[0]), qv[i][1] * fast_exp2(b[i][1] - ref_q[1]), hi, lo);
+          split2(qv[i][0] * fast_exp2(b.x - ref_q[0]), qv[i][1] * fast_exp2(b.y - ref_q[1]), hi, lo);
           *reinterpret_cast<uint32_t*>(sm + T_Q + at) = hi;
           *reinterpret_cast<uint32_t*>(sm + T_Q + T_SPLIT + at) = lo;
         }
       }
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int j = tid + i * LC_THREADS, t = j >> 4, col = (j & 15) * 8;
-        if (col < V) *reinterpret_cast<uint4*>(sm + T_V + pair_at(t, col, LC)) = vv[i];
-      }
       fence_proxy_async_smem();
       tc_fence_before();
       mbar_arrive_warp(b_qk);
-      lc_meet();                                          // references and factors
+      mbar_arrive_warp(b_free);
+      lc_meet();                                          // factors of the state
       // ---- state: operand of the product with Q, and the sum that K^T V is added to
       {
-        uint32_t r[32];
+        uint32_t r[32], hi[16], lo[16];
         __syncwarp();
         tmem_ld32(tmem + TM_S + lanes + cg * 32, r);
         tmem_ld_wait();
-        const float f = exp2f(pend[(n & 1) * 128 + srow]), fq = exp2f(rq[srow]), fk = exp2f(rk[srow]);
 #pragma unroll
-        for (int j = 0; j < 32; j += 8) {
-          float s[8];
-          uint32_t hi[4], lo[4];
-#pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            s[e] = __uint_as_float(r[j + e]) * f;
-            r[j + e] = __float_as_uint(s[e] * fk);
-            s[e] *= fq;
-          }
+        for (int j = 0; j < 32; j += 4) {
+          const float4 w0 = *reinterpret_cast<const float4*>(f0 + cg * 32 + j), wk = *reinterpret_cast<const float4*>(fk + cg * 32 + j);
+          const float x0 = __uint_as_float(r[j]) * w0.x, x1 = __uint_as_float(r[j + 1]) * w0.y, x2 = __uint_as_float(r[j + 2]) * w0.z,
+                      x3 = __uint_as_float(r[j + 3]) * w0.w;
+          const float y0 = x0 * wk.x, y1 = x1 * wk.y, y2 = x2 * wk.z, y3 = x3 * wk.w;
           if (OUT) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) split2(s[2 * e], s[2 * e + 1], hi[e], lo[e]);
-            const uint32_t at = T_S + pair_at(srow, cg * 32 + j, 128);
-            *reinterpret_cast<uint4*>(sm + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-            *reinterpret_cast<uint4*>(sm + at + 32768) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            split2(far ? x0 : y0, far ? x1 : y1, hi[j / 2], lo[j / 2]);
+            split2(far ? x2 : y2, far ? x3 : y3, hi[j / 2 + 1], lo[j / 2 + 1]);
           }
+          r[j] = __float_as_uint(y0);
+          r[j + 1] = __float_as_uint(y1);
+          r[j + 2] = __float_as_uint(y2);
+          r[j + 3] = __float_as_uint(y3);
         }
         __syncwarp();
         tmem_st32(tmem + TM_S + lanes + cg * 32, r);
+        if (OUT) {
+          tmem_st16(tmem + TM_SH + lanes + cg * 16, hi);
+          tmem_st16(tmem + TM_SL + lanes + cg * 16, lo);
+        }
         tmem_st_wait();
       }
-      if (OUT && quad < 2 && !far) {
-        // ---- A, lower triangle, as two bf16 parts
+      if (OUT && !far) {
+        // ---- A, lower triangle: the quarters of Qh (lanes 0 .. 63) as two bf16 parts, those of Ql as one
         ok &= mbar_wait(bar_a, n & 1, dead, c.status, 800);
         tc_fence_after();
-        const int t = srow;
-        uint32_t r[16];
+        const int t = lrow & 63;
+        uint32_t r[16], r2[16];
         __syncwarp();
         tmem_ld16(tmem + TM_A + lanes + cg * 16, r);
+        tmem_ld16(tmem + TM_A + LC + lanes + cg * 16, r2);
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 16; j += 8) {
           uint32_t hi[4], lo[4];
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const int s = cg * 16 + j + 2 * e;
-            split2(s <= t ? __uint_as_float(r[j + 2 * e]) : 0.0f, s + 1 <= t ? __uint_as_float(r[j + 2 * e + 1]) : 0.0f, hi[e], lo[e]);
+            const int i = j + 2 * e, s = cg * 16 + i;
+            split2(s <= t ? __uint_as_float(r[i]) + __uint_as_float(r2[i]) : 0.0f,
+                   s + 1 <= t ? __uint_as_float(r[i + 1]) + __uint_as_float(r2[i + 1]) : 0.0f, hi[e], lo[e]);
           }
-          const uint32_t at = T_A + sw128_offset(t, (cg * 16 + j) >> 3);
-          *reinterpret_cast<uint4*>(sm + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(sm + at + 8192) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          const uint32_t at = sw128_offset(t, (cg * 16 + j) >> 3);
+          *reinterpret_cast<uint4*>(sm + (quad < 2 ? T_A : T_A2) + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          if (quad < 2) *reinterpret_cast<uint4*>(sm + T_A + T_SPLIT + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
       }
       fence_proxy_async_smem();
       tc_fence_before();
       mbar_arrive_warp(b_sa);
       if (n + 1 < n_chunks) gates(n + 1);                 // while the tensor core works
-      if (OUT && quad < 2) {
-        // ---- result: lane = token, this warp's 32 columns; norm over the head, gate
+      if (OUT) {
+        // ---- result: lane = element of v, this warp's 16 tokens; norm over the head, gate.  Rows go through the tile of Q
+        // (its products are done) to leave in 16-byte pieces.
+        uint4 g[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          g[i] = make_uint4(0, 0, 0, 0);
+          if (a.gate && o_mine && o_row + 8 * i < left) g[i] = *reinterpret_cast<const uint4*>(gp + (long long)(t0 + o_row + 8 * i) * a.ldg);
+        }
         ok &= mbar_wait(bar_o, n & 1, dead, c.status, 801);
         tc_fence_after();
-        const int t = srow;
-        uint32_t r[32];
-        __syncwarp();
-        tmem_ld32(tmem + TM_O + lanes + cg * 32, r);
-        tmem_ld_wait();
-        float ss = 0.0f;
+        float* rows = reinterpret_cast<float*>(sm + T_Q);
+        {
+          float sq[16];
+          uint32_t r[16], r2[16];
+          __syncwarp();
+          tmem_ld16(tmem + TM_O + lanes + cg * 16, r);
+          tmem_ld16(tmem + TM_O + LC + lanes + cg * 16, r2);
+          tmem_ld_wait();
+          tc_fence_before();
 #pragma unroll
-        for (int j = 0; j < 32; ++j) ss = fmaf(__uint_as_float(r[j]), __uint_as_float(r[j]), ss);
-        red[cg * LC + t] = ss;
-        asm volatile("bar.sync 2, 256;" ::: "memory");
-        if (t < left) {
-          const float rs = 1.0f / sqrtf((red[t] + red[LC + t] + red[2 * LC + t] + red[3 * LC + t]) / V + a.eps);
-          const long long row = t0 + t;
-          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(a.out) + (row0 + row) * a.ldo + (long long)h * V + cg * 32;
-          const __nv_bfloat16* g = gp + row * a.ldg + cg * 32;
-#pragma unroll
-          for (int j = 0; j < 32; j += 8) {
-            if (cg * 32 + j >= V) continue;
-            float x[8];
-#pragma unroll
-            for (int e = 0; e < 8; e += 4) {
-              const float4 w = *reinterpret_cast<const float4*>(a.w + cg * 32 + j + e);
-              x[e] = __uint_as_float(r[j + e]) * rs * w.x;
-              x[e + 1] = __uint_as_float(r[j + e + 1]) * rs * w.y;
-              x[e + 2] = __uint_as_float(r[j + e + 2]) * rs * w.z;
-              x[e + 3] = __uint_as_float(r[j + e + 3]) * rs * w.w;
-            }
-            if (a.gate) {
-              const uint4 u = *reinterpret_cast<const uint4*>(g + j);
-              const uint32_t gu[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                const float2 f = unpack_bf16x2(gu[e]);
-                x[2 * e] *= lin_silu_fast(f.x);
-                x[2 * e + 1] *= lin_silu_fast(f.y);
-              }
-            }
-            *reinterpret_cast<uint4*>(o + j) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+          for (int j = 0; j < 16; ++j) {
+            const float o = __uint_as_float(r[j]) + __uint_as_float(r2[j]);
+            rows[(cg * 16 + j) * 128 + lrow] = o;
+            sq[j] = lrow < V ? o * o : 0.0f;              // lanes behind the head hold other columns of the rows
           }
+          const float mine_sum = sum_over_lanes(sq, lane);
+          if ((lane & 1) == 0) red[quad * LC + cg * 16 + (lane >> 1)] = mine_sum;
         }
-        tc_fence_before();
+        asm volatile("bar.sync %0, 128;" ::"r"(2 + cg) : "memory");
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int t = o_row + 8 * i;
+          if (!o_mine || t >= left) continue;
+          const float scale = 1.0f / sqrtf((red[t] + red[LC + t] + red[2 * LC + t] + red[3 * LC + t]) / V + a.eps);
+          const float4 x0 = *reinterpret_cast<const float4*>(rows + t * 128 + o_col), x1 = *reinterpret_cast<const float4*>(rows + t * 128 + o_col + 4);
+          const float4 w0 = *reinterpret_cast<const float4*>(a.w + o_col), w1 = *reinterpret_cast<const float4*>(a.w + o_col + 4);
+          float x[8] = {x0.x * scale * w0.x, x0.y * scale * w0.y, x0.z * scale * w0.z, x0.w * scale * w0.w,
+                        x1.x * scale * w1.x, x1.y * scale * w1.y, x1.z * scale * w1.z, x1.w * scale * w1.w};
+          if (a.gate) {
+            const uint32_t gu[4] = {g[i].x, g[i].y, g[i].z, g[i].w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 f = unpack_bf16x2(gu[e]);
+              x[2 * e] *= lin_silu_fast(f.x);
+              x[2 * e + 1] *= lin_silu_fast(f.y);
+            }
+          }
+          *reinterpret_cast<uint4*>(op + (long long)(t0 + t) * a.ldo) =
+              make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+        }
       }
     }
     // ---- last state: to the cache, or as the stretch's sum
     if (n_chunks > 0) ok &= mbar_wait(bar_s, (n_chunks - 1) & 1, dead, c.status, 803);
     tc_fence_after();
+    lc_meet();
+    if (tg == 0) { f0[ch] = exp2f(pend[0]); f0[ch + 1] = exp2f(pend[1]); }
+    lc_meet();
     if (ok && (!OUT || last)) {
       uint32_t r[32];
       __syncwarp();
       tmem_ld32(tmem + TM_S + lanes + cg * 32, r);
       tmem_ld_wait();
-      const float f = exp2f(pend[(n_chunks & 1) * 128 + srow]);
       float* dst = OUT ? a.state + ((slot * a.history + (p0 + count) % a.history) * a.heads + h) * (long long)D * V
                        : c.start + ((long long)blockIdx.y * a.heads + h) * D * V;
-      if (srow < D) {
 #pragma unroll
-        for (int j = 0; j < 32; j += 4)
-          if (cg * 32 + j < V) {
-            const float v[4] = {__uint_as_float(r[j]) * f, __uint_as_float(r[j + 1]) * f, __uint_as_float(r[j + 2]) * f, __uint_as_float(r[j + 3]) * f};
-            stv<4>(dst + (long long)srow * V + cg * 32 + j, v);
-          }
+      for (int j = 0; j < 32; ++j)
+        if (lrow < V && cg * 32 + j < D) dst[(long long)(cg * 32 + j) * V + lrow] = __uint_as_float(r[j]) * f0[cg * 32 + j];
+      if (!OUT && tg == 0 && mine) {
+        float* total = c.total + ((long long)blockIdx.y * a.heads + h) * D + ch;
+        total[0] = tot[0];
+        total[1] = tot[1];
       }
-      if (!OUT && tid < D) c.total[((long long)blockIdx.y * a.heads + h) * D + tid] = tot[tid];
     }
   }
   if (*dead) __nanosleep(100000);
@@ -483,7 +478,7 @@ linear_chunks_kernel(const ChunksDev c) {
   __syncthreads();
   if (warp == 0) {
     tc_fence_after();
-    tmem_dealloc(tmem, COLS);
+    tmem_dealloc(tmem, 512);
   }
 }
 
@@ -522,9 +517,9 @@ CGK_API int cgk_linear_chunks_ok(int D, int V) { return D % 8 == 0 && V % 8 == 0
 
 CGK_API long long cgk_linear_chunks_scratch_floats(int n_items, int heads, int D, int V) { return (long long)n_items * heads * D * (V + 1); }
 
-CGK_API int cgk_linear_chunks(const cgk_linear_state_args* pa, const int* items, int n_items, const int* run_items, int n_runs, void* scratch,
-                              void* stream) {
-  CGK_REQUIRE(pa && items && n_items >= 0 && (!scratch || (run_items && n_runs > 0)), "cgk_linear_chunks: bad arguments");
+CGK_API int cgk_linear_chunks(const cgk_linear_state_args* pa, int n_rows, const int* items, int n_items, const int* run_items, int n_runs,
+                              void* scratch, void* stream) {
+  CGK_REQUIRE(pa && items && n_rows > 0 && n_items >= 0 && (!scratch || (run_items && n_runs > 0)), "cgk_linear_chunks: bad arguments");
   const cgk_linear_state_args& a = *pa;
   CGK_REQUIRE(a.q && a.v && a.z && a.bias && a.w && a.state && a.out && a.slot && a.pos && a.heads > 0 && a.history > 0 && a.slots > 0 && !a.fp32,
               "cgk_linear_chunks: bad arguments");
@@ -547,18 +542,29 @@ CGK_API int cgk_linear_chunks(const cgk_linear_state_args* pa, const int* items,
   const dim3 grid(a.heads, n_items);
   auto sums = a.mode == GATE_BOUNDED ? linear_chunks_kernel<false, GATE_BOUNDED> : linear_chunks_kernel<false, GATE_ROOT>;
   auto results = a.mode == GATE_BOUNDED ? linear_chunks_kernel<true, GATE_BOUNDED> : linear_chunks_kernel<true, GATE_ROOT>;
-  if (scratch) {
-    const int smem = T_END_SUM + LC_MISC + 1024;
-    CGK_CUDA_CHECK(cudaFuncSetAttribute(sums, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    sums<<<grid, LC_THREADS + 32, smem, st>>>(d);
+  // rows as the kernels read them: all tokens of the call, one head's columns at a time
+  CUtensorMap tz, tq, tk, tv;
+  auto rows_map = [&](CUtensorMap* m, const void* p, bool fp32, long long ld, int width, int box_cols, Swz swz) {
+    const int es = fp32 ? 4 : 2;
+    uint64_t dims[2] = {(uint64_t)width, (uint64_t)n_rows}, strides[1] = {(uint64_t)ld * es};
+    uint32_t box[2] = {(uint32_t)box_cols, LC};
+    return encode_tmap(m, p, fp32 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dims, strides, box, swz);
+  };
+  int rc;
+  if ((rc = rows_map(&tz, a.z, true, a.ldz, a.heads * a.D, a.D, Swz::None)) || (rc = rows_map(&tq, a.q, false, a.ldq, a.heads * a.D, a.D, Swz::None)) ||
+      (rc = rows_map(&tk, a.k ? a.k : a.q, false, a.k ? a.ldk : a.ldq, a.heads * a.D, a.D, Swz::None)) ||
+      (rc = rows_map(&tv, a.v, false, a.ldv, a.heads * a.V, 64, Swz::B128)))
+    return rc;
+  for (auto kernel : {scratch ? sums : nullptr, results}) {
+    if (!kernel) continue;
+    CGK_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LC_SMEM));
+    kernel<<<grid, LC_THREADS + 128, LC_SMEM, st>>>(tz, tq, tk, tv, d);
     CGK_LAUNCH_CHECK();
-    linear_starts_kernel<<<dim3((a.D * a.V / 4 + 255) / 256, a.heads, n_runs), 256, 0, st>>>(d, run_items);
-    CGK_LAUNCH_CHECK();
+    if (kernel == sums) {
+      linear_starts_kernel<<<dim3((a.D * a.V / 4 + 255) / 256, a.heads, n_runs), 256, 0, st>>>(d, run_items);
+      CGK_LAUNCH_CHECK();
+    }
   }
-  const int smem = T_END + LC_MISC + 1024;
-  CGK_CUDA_CHECK(cudaFuncSetAttribute(results, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  results<<<grid, LC_THREADS + 32, smem, st>>>(d);
-  CGK_LAUNCH_CHECK();
   return 0;
 }
 

@@ -139,14 +139,6 @@ __device__ __forceinline__ uint32_t mbar_try_wait_suspend(uint32_t bar, uint32_t
   return ok;
 }
 
-// Asynchronous copy global -> shared of 4 or 8 bytes per thread (both addresses aligned to that).
-template <int BYTES>
-__device__ __forceinline__ void cp_async(uint32_t dst_smem, const void* src) {
-  static_assert(BYTES == 4 || BYTES == 8, "4 or 8 bytes");
-  asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(dst_smem), "l"(src), "n"(BYTES) : "memory");
-}
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
-
 // Untiled bulk copy global -> shared, completing on an mbarrier.  Both addresses 16-byte aligned,
 // `bytes` a multiple of 16.
 __device__ __forceinline__ void bulk_load_1d(uint32_t dst_smem, const void* src, uint32_t bytes, uint32_t bar) {
@@ -404,6 +396,16 @@ __device__ __forceinline__ void umma_f16_lane(uint32_t mine, uint32_t d_tmem, ui
       "setp.ne.b32 m, %5, 0;\n\t"
       "@m tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
       ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(mine)
+      : "memory");
+}
+__device__ __forceinline__ void umma_f16_ts_lane(uint32_t mine, uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc,
+                                                 uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, m;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "setp.ne.b32 m, %5, 0;\n\t"
+      "@m tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      ::"r"(d_tmem), "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(mine)
       : "memory");
 }
 __device__ __forceinline__ void umma_commit_lane(uint32_t mine, uint32_t bar) {

@@ -387,9 +387,10 @@ typedef struct {
 } cgk_linear_state_args;
 int cgk_linear_state(const cgk_linear_state_args* a, int n_runs, void* stream);
 /* The same over stretches of 64-token chunks on the tensor cores (bf16 rows, D and V multiples of 8 up to 128, 16-byte aligned rows; `runs` is
- * not used).  items [n_items][4]: first row, tokens, run, 1 for the last stretch of its run; the stretches of a run in order, all but the last
+ * not used); n_rows rows exist.  items [n_items][4]: first row, tokens, run, 1 for the last stretch of its run; the stretches of a run in order, all but the last
  * a multiple of 64 tokens.  scratch null: every run is one stretch; otherwise run_items [n_runs][2] = first item and number of items. */
-int cgk_linear_chunks(const cgk_linear_state_args* a, const int* items, int n_items, const int* run_items, int n_runs, void* scratch, void* stream);
+int cgk_linear_chunks(const cgk_linear_state_args* a, int n_rows, const int* items, int n_items, const int* run_items, int n_runs, void* scratch,
+                      void* stream);
 int cgk_linear_chunks_ok(int D, int V);
 long long cgk_linear_chunks_scratch_floats(int n_items, int heads, int D, int V);
 
