@@ -8,6 +8,8 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
+#include "sm100.cuh"
+
 namespace cgk {
 
 enum : int { GATE_BOUNDED = 0, GATE_ROOT = 1 };
@@ -56,32 +58,44 @@ __device__ __forceinline__ float lin_lg2(float x) {
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// two channels at once, in packed fp32 arithmetic
+struct Pair { float x, y; };
+__device__ __forceinline__ Pair pfma(Pair a, Pair b, Pair c) { Pair d; ffma2(d.x, d.y, a.x, a.y, b.x, b.y, c.x, c.y); return d; }
+__device__ __forceinline__ Pair pmul(Pair a, Pair b) { Pair d; fmul2(d.x, d.y, a.x, a.y, b.x, b.y); return d; }
+__device__ __forceinline__ Pair padd(Pair a, Pair b) { fadd2(a.x, a.y, b.x, b.y); return a; }
+__device__ __forceinline__ Pair pall(float v) { return Pair{v, v}; }
+// y: gate with its bias; low: lower bounds; returns the logarithms, *key the keys of GATE_BOUNDED
 template <int MODE>
-__device__ __forceinline__ float lin_decay_log2(float y, float low, float inv_tau, float* one_minus) {
+__device__ __forceinline__ Pair lin_decay_log2(Pair y, Pair low, float inv_tau, Pair* key) {
   constexpr float LOG2E = 1.4426950408889634f;
-  const float e = lin_ex2(-fabsf(y) * LOG2E);
-  if constexpr (MODE == GATE_ROOT) {                       // -(max(-y, 0) log2 e + log2(1 + e)) / tau
-    const float u = e * lin_rcp(2.0f + e), u2 = u * u;
-    float p = fmaf(u2, 1.0f / 15, 1.0f / 13);
-    p = fmaf(u2, p, 1.0f / 11);
-    p = fmaf(u2, p, 1.0f / 9);
-    p = fmaf(u2, p, 1.0f / 7);
-    p = fmaf(u2, p, 1.0f / 5);
-    p = fmaf(u2, p, 1.0f / 3);
-    p = fmaf(u2 * u, p, u);
-    return fmaf(p, -2.0f * LOG2E, fminf(y, 0.0f) * LOG2E) * inv_tau;
+  const Pair e = {lin_ex2(-fabsf(y.x) * LOG2E), lin_ex2(-fabsf(y.y) * LOG2E)};
+  if constexpr (MODE == GATE_ROOT) {                       // -(max(-y, 0) log2 e + log2(1 + e)) / tau, u = e / (2 + e) <= 1/3
+    const Pair d = padd(e, pall(2.0f)), u = pmul(e, Pair{lin_rcp(d.x), lin_rcp(d.y)}), u2 = pmul(u, u);
+    Pair p = pfma(u2, pall(1.0f / 13), pall(1.0f / 11));
+    p = pfma(u2, p, pall(1.0f / 9));
+    p = pfma(u2, p, pall(1.0f / 7));
+    p = pfma(u2, p, pall(1.0f / 5));
+    p = pfma(u2, p, pall(1.0f / 3));
+    p = pfma(pmul(u2, u), p, u);
+    const Pair m = {fminf(y.x, 0.0f), fminf(y.y, 0.0f)};
+    return pfma(p, pall(-2.0f * LOG2E * inv_tau), pmul(m, pall(LOG2E * inv_tau)));
   } else {
     // one reciprocal for 1 / (1 + e) and for u = k / (2 - k), k = room * num / (1 + e)
-    const float room = 1.0f - low, num = y >= 0.0f ? e : 1.0f, one = 1.0f + e, rn = room * num, den = fmaf(2.0f, one, -rn);
-    const float r = lin_rcp(one * den), inv = r * den, k = rn * inv, f = fmaf(room * inv, y >= 0.0f ? 1.0f : e, low);
-    *one_minus = k;
-    const float u = rn * one * r, u2 = u * u;               // k <= 1/4: u <= 1/7
-    float p = fmaf(u2, 1.0f / 9, 1.0f / 7);
-    p = fmaf(u2, p, 1.0f / 5);
-    p = fmaf(u2, p, 1.0f / 3);
-    p = fmaf(u2 * u, p, u);
-    return k <= 0.25f ? p * (-2.0f * LOG2E) : lin_lg2(fmaxf(f, 1e-37f));
+    const bool px = y.x >= 0.0f, py = y.y >= 0.0f;
+    const Pair room = padd(pall(1.0f), Pair{-low.x, -low.y}), num = {px ? e.x : 1.0f, py ? e.y : 1.0f}, rest = {px ? 1.0f : e.x, py ? 1.0f : e.y};
+    const Pair one = padd(e, pall(1.0f)), rn = pmul(room, num), den = pfma(one, pall(2.0f), Pair{-rn.x, -rn.y}), od = pmul(one, den);
+    const Pair r = {lin_rcp(od.x), lin_rcp(od.y)}, inv = pmul(r, den), k = pmul(rn, inv), f = pfma(pmul(room, inv), rest, low);
+    const Pair u = pmul(rn, pmul(one, r)), u2 = pmul(u, u);   // k <= 1/4: u <= 1/7
+    Pair p = pfma(u2, pall(1.0f / 7), pall(1.0f / 5));
+    p = pfma(u2, p, pall(1.0f / 3));
+    p = pmul(pfma(pmul(u2, u), p, u), pall(-2.0f * LOG2E));
+    *key = k;
+    return Pair{k.x <= 0.25f ? p.x : lin_lg2(fmaxf(f.x, 1e-37f)), k.y <= 0.25f ? p.y : lin_lg2(fmaxf(f.y, 1e-37f))};
   }
+}
+__device__ __forceinline__ Pair lin_silu_fast(Pair x) {
+  const Pair t = pmul(x, pall(-1.4426950408889634f)), d = padd(Pair{lin_ex2(t.x), lin_ex2(t.y)}, pall(1.0f));
+  return pmul(x, Pair{lin_rcp(d.x), lin_rcp(d.y)});
 }
 __device__ __forceinline__ float lin_silu_fast(float x) { return x * lin_rcp(1.0f + lin_ex2(-1.4426950408889634f * x)); }
 

@@ -40,8 +40,8 @@ struct ChunksDev {
 
 __device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x0, x1);
-  const float2 h = unpack_bf16x2(hi);
-  lo = pack_bf16x2(x0 - h.x, x1 - h.y);
+  const Pair rest = pfma(Pair{__uint_as_float(hi << 16), __uint_as_float(hi & 0xffff0000u)}, pall(-1.0f), Pair{x0, x1});
+  lo = pack_bf16x2(rest.x, rest.y);
 }
 // byte offset of a 4-byte pair of columns in a tile with `rows` rows per block
 __device__ __forceinline__ uint32_t pair_at(int row, int col, int rows) {
@@ -126,14 +126,14 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
   const uint32_t tmem = *tmem_slot;
   // 640 threads are launched with 96 registers each; the last warpgroup leaves some of its share to the workers
   if (warp >= 16) {
-    asm volatile("setmaxnreg.dec.sync.aligned.u32 56;");
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 32;");
    if (warp == 17) {
     // ------------------------------ loader ------------------------------
     // 64 rows at a time; what lies behind the end of the run is another run's (or zero) and is not used
     if (lane == 0) {
       const int v_blocks = (V + 63) / 64;
       for (int n = 0; n < n_chunks; ++n) {
-        const int row = row0 + n * LC;
+        const int row = row0 + (OUT ? n : n_chunks - 1 - n) * LC;
         if (n > 0 && !mbar_wait(b_free, (n - 1) & 1, dead, c.status, 820)) break;
         mbar_expect_tx(b_raw, LC * D * (4 + (OUT ? 2 : 0) + (MODE == GATE_ROOT ? 2 : 0)));
         tma_load_2d(sb + R_Z, &tm_z, b_raw, h * D, row);
@@ -185,22 +185,22 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
       }
 #pragma unroll
       for (int kk = 0; kk < 2 * LC / 16; ++kk)
-        umma_f16_lane(mine, tm + TM_S, mn_major(dv, kk & 3), mn_major(dkt + (kk >= 4 ? T_SPLIT >> 4 : 0), kk & 3), id_mm, 1);
+        umma_f16_lane(mine, tm + TM_S, mn_major(dv, kk & 3), mn_major(dkt + (kk >= 4 ? T_SPLIT >> 4 : 0), kk & 3), id_mm, OUT || n > 0 || kk > 0);
       umma_commit_lane(mine, bar_s);
     }
    }
   } else {
-    asm volatile("setmaxnreg.inc.sync.aligned.u32 104;");
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 112;");
     // ------------------------------ workers ------------------------------
     const int quad = warp & 3, cg = warp >> 2, lrow = quad * 32 + lane;       // TMEM lane: an element of v, or a row of A
     const uint32_t lanes = (uint32_t)(quad * 32) << 16;
     const int p0 = a.pos[row0];
     const long long slot = CGK_IDX(a.slot[row0], a.slots);
-    {
+    if (OUT) {
       // first state -> TMEM: this warp's 32 state rows
       const float* src = nullptr;
-      if (OUT && c.start) src = c.start + ((long long)blockIdx.y * a.heads + h) * D * V;
-      else if (OUT && p0 > 0) src = a.state + ((slot * a.history + p0 % a.history) * a.heads + h) * (long long)D * V;
+      if (c.start) src = c.start + ((long long)blockIdx.y * a.heads + h) * D * V;
+      else if (p0 > 0) src = a.state + ((slot * a.history + p0 % a.history) * a.heads + h) * (long long)D * V;
       uint32_t r[32];
 #pragma unroll
       for (int j = 0; j < 32; ++j)
@@ -211,45 +211,43 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
     // results leave with two 16-byte pieces per thread: rows cg * 16 + (0, 8) + .., columns o_col ..
     const int o_row = cg * 16 + (quad * 32 + lane) / 16, o_col = (lane & 15) * 8;
     const bool o_mine = o_col < V;
+    const float inv_v = 1.0f / V;
     const __nv_bfloat16* gp = reinterpret_cast<const __nv_bfloat16*>(a.gate) + (a.gate ? (long long)row0 * a.ldg + h * V + o_col : 0);
     __nv_bfloat16* op = reinterpret_cast<__nv_bfloat16*>(a.out) + (long long)row0 * a.ldo + h * V + o_col;
     const int ch = (tid & 63) * 2, tg = tid >> 6;         // two state rows, eight tokens
     const bool mine = ch < D;
-    const float bias0 = mine ? a.bias[h * D + ch] : 0.0f, bias1 = mine ? a.bias[h * D + ch + 1] : 0.0f;
-    const float low0 = MODE == GATE_BOUNDED && mine ? a.low[h * D + ch] : 0.0f, low1 = MODE == GATE_BOUNDED && mine ? a.low[h * D + ch + 1] : 0.0f;
+    const Pair bias = mine ? Pair{a.bias[h * D + ch], a.bias[h * D + ch + 1]} : pall(0.0f);
+    const Pair low = MODE == GATE_BOUNDED && mine ? Pair{a.low[h * D + ch], a.low[h * D + ch + 1]} : pall(0.0f);
     bool ok = true;                                       // after a wait that ran out a warp still comes to every meeting point
 
-    float kv[8][2], qv[8][2], pend[2] = {0.0f, 0.0f}, tot[2] = {0.0f, 0.0f};
-    auto gates = [&](int n) {                             // decays and their sums over eight tokens, keys, queries
-      ok &= mbar_wait(b_raw, n & 1, dead, c.status, 821);
-      float sum0 = 0.0f, sum1 = 0.0f;
+    Pair kv[8], qv[8], pend = pall(0.0f), tot = pall(0.0f);
+    auto gates = [&](int n, int at) {                     // the n-th chunk of the loop is the at-th of the stretch: decays
+      ok &= mbar_wait(b_raw, n & 1, dead, c.status, 821);  // and their sums over eight tokens, keys, queries
+      Pair sum = pall(0.0f);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int t = tg * 8 + i;
-        const bool in = mine && n * LC + t < count;       // otherwise the place holds an earlier chunk's row
-        const float2 z = in ? *reinterpret_cast<const float2*>(sm + R_Z + (t * D + ch) * 4) : make_float2(0.0f, 0.0f);
-        float k0 = 0.0f, k1 = 0.0f;
-        const float g0 = lin_decay_log2<MODE>(z.x + bias0, low0, a.inv_tau, &k0);
-        const float g1 = lin_decay_log2<MODE>(z.y + bias1, low1, a.inv_tau, &k1);
+        const bool in = mine && at * LC + t < count;      // what lies behind the run does not count
+        Pair* place = reinterpret_cast<Pair*>(sm + R_Z + (t * D + (mine ? ch : 0)) * 4);
+        Pair k = pall(0.0f);
+        const Pair g = lin_decay_log2<MODE>(padd(*place, bias), low, a.inv_tau, &k);
         if (MODE == GATE_ROOT) {
-          const float2 k = unpack_bf16x2(in ? *reinterpret_cast<const uint32_t*>(sm + R_X + (t * D + ch) * 2) : 0u);
-          k0 = k.x;
-          k1 = k.y;
+          const float2 w = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(sm + R_X + (t * D + (mine ? ch : 0)) * 2));
+          k = Pair{w.x, w.y};
         }
-        kv[i][0] = in ? k0 : 0.0f;
-        kv[i][1] = in ? k1 : 0.0f;
+        kv[i] = Pair{in ? k.x : 0.0f, in ? k.y : 0.0f};
         if (OUT) {
-          const float2 q = unpack_bf16x2(in ? *reinterpret_cast<const uint32_t*>(sm + R_W + (t * D + ch) * 2) : 0u);
-          qv[i][0] = (a.q_silu ? lin_silu_fast(q.x) : q.x) * a.q_scale;
-          qv[i][1] = (a.q_silu ? lin_silu_fast(q.y) : q.y) * a.q_scale;
+          const float2 w = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(sm + R_W + (t * D + (mine ? ch : 0)) * 2));
+          const Pair q = {in ? w.x : 0.0f, in ? w.y : 0.0f};
+          qv[i] = pmul(a.q_silu ? lin_silu_fast(q) : q, pall(a.q_scale));
         }
-        sum0 += in ? g0 : 0.0f;
-        sum1 += in ? g1 : 0.0f;
-        if (mine) *reinterpret_cast<float2*>(sm + R_Z + (t * D + ch) * 4) = make_float2(sum0, sum1);      // read back by this thread
+        sum = padd(sum, Pair{in ? g.x : 0.0f, in ? g.y : 0.0f});
+        if (mine) *place = sum;                           // read back by this thread
       }
-      *reinterpret_cast<float2*>(part + tg * 128 + ch) = make_float2(sum0, sum1);
+      *reinterpret_cast<Pair*>(part + tg * 128 + ch) = sum;
     };
-    gates(0);
+    auto chunk_of = [&](int n) { return OUT ? n : n_chunks - 1 - n; };      // the sums are taken from the end
+    if (n_chunks > 0) gates(0, chunk_of(0));
 
     for (int n = 0; n < n_chunks; ++n) {
       const int t0 = n * LC, left = min(LC, count - t0);
@@ -257,21 +255,19 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
       if (n > 0) ok &= mbar_wait(bar_s, (n - 1) & 1, dead, c.status, 802);
       tc_fence_after();
       lc_meet();
-      float before[2] = {0.0f, 0.0f}, mid[2] = {0.0f, 0.0f}, end[2] = {0.0f, 0.0f};
+      Pair before = pall(0.0f), mid = pall(0.0f), end = pall(0.0f);
 #pragma unroll
       for (int g = 0; g < 8; ++g) {
-        const float2 s = *reinterpret_cast<const float2*>(part + g * 128 + ch);
-        if (g == tg) { before[0] = end[0]; before[1] = end[1]; }
-        end[0] += s.x;
-        end[1] += s.y;
-        if (g == 3) { mid[0] = end[0]; mid[1] = end[1]; }
+        const Pair s = *reinterpret_cast<const Pair*>(part + g * 128 + ch);
+        if (g == tg) before = end;
+        end = padd(end, s);
+        if (g == 3) mid = end;
       }
       auto sum_at = [&](int i) {                          // decay up to and with this thread's token i
-        const float2 s = mine ? *reinterpret_cast<const float2*>(sm + R_Z + ((tg * 8 + i) * D + ch) * 4) : make_float2(0.0f, 0.0f);
-        return make_float2(s.x + before[0], s.y + before[1]);
+        return mine ? padd(*reinterpret_cast<const Pair*>(sm + R_Z + ((tg * 8 + i) * D + ch) * 4), before) : pall(0.0f);
       };
       bool far = false;
-      if (OUT) far = lc_any(fmaxf(-mid[0], -mid[1]) > LC_LIMIT || fmaxf(mid[0] - end[0], mid[1] - end[1]) > LC_LIMIT);
+      if (OUT) far = lc_any(fmaxf(-mid.x, -mid.y) > LC_LIMIT || fmaxf(mid.x - end.x, mid.y - end.y) > LC_LIMIT);
       if (far) {
         // A term by term: row tid / 8, columns 8 (tid % 8) ..; scratch space: the tiles of Q and K, and b in its own rows
         float* fx = reinterpret_cast<float*>(sm + T_Q);
@@ -280,11 +276,11 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const int at = (tg * 8 + i) * 128 + ch;
-          *reinterpret_cast<float2*>(fx + at) = make_float2(qv[i][0], qv[i][1]);
-          *reinterpret_cast<float2*>(fy + at) = make_float2(kv[i][0], kv[i][1]);
-          if (mine) *reinterpret_cast<float2*>(fb + (tg * 8 + i) * D + ch) = sum_at(i);
+          *reinterpret_cast<Pair*>(fx + at) = qv[i];
+          *reinterpret_cast<Pair*>(fy + at) = kv[i];
+          if (mine) *reinterpret_cast<Pair*>(fb + (tg * 8 + i) * D + ch) = sum_at(i);
         }
-        before[0] = before[1] = 0.0f;                     // b's rows are complete now
+        before = pall(0.0f);                              // b's rows are complete now
         lc_meet();
         const int t = tid >> 3, s0 = (tid & 7) * 8;
         uint32_t hi[4], lo[4];
@@ -306,42 +302,44 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
         *reinterpret_cast<uint4*>(sm + T_A + T_SPLIT + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         *reinterpret_cast<uint4*>(sm + T_A2 + at) = make_uint4(0, 0, 0, 0);
       }
-      const float ref_q[2] = {far ? 0.0f : mid[0], far ? 0.0f : mid[1]};
-      const float ref_k[2] = {far || !OUT ? end[0] : mid[0], far || !OUT ? end[1] : mid[1]};
-      if (tg == 0) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          f0[ch + i] = exp2f(pend[i]);
-          fk[ch + i] = exp2f(ref_k[i]);                   // Q's reference is the same, or 0
-        }
+      // K's factors refer to the chunk's middle or end; the summing pass comes from the end and adds what follows
+      const Pair ref_q = far ? pall(0.0f) : mid, ref_k = OUT ? (far ? end : mid) : padd(end, tot);
+      if (OUT && tg == 0) {
+        f0[ch] = exp2f(pend.x);
+        f0[ch + 1] = exp2f(pend.y);
+        fk[ch] = exp2f(ref_k.x);                          // Q's reference is the same, or 0
+        fk[ch + 1] = exp2f(ref_k.y);
         if (tid == 0) *far_flag = far;
       }
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        pend[i] = end[i] - ref_k[i];
-        tot[i] += end[i];
-      }
+      pend = padd(end, Pair{-ref_k.x, -ref_k.y});
+      tot = padd(tot, end);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const uint32_t at = pair_at(tg * 8 + i, ch, 128);
-        const float2 b = sum_at(i);
+        const Pair b = sum_at(i), bk = pfma(b, pall(-1.0f), ref_k);
         uint32_t hi, lo;
-        split2(kv[i][0] * fast_exp2(ref_k[0] - b.x), kv[i][1] * fast_exp2(ref_k[1] - b.y), hi, lo);
+        const Pair k = pmul(kv[i], Pair{fast_exp2(bk.x), fast_exp2(bk.y)});
+        split2(k.x, k.y, hi, lo);
         *reinterpret_cast<uint32_t*>(sm + T_K + at) = hi;
         *reinterpret_cast<uint32_t*>(sm + T_K + T_SPLIT + at) = lo;
         if (OUT) {
-          split2(qv[i][0] * fast_exp2(b.x - ref_q[0]), qv[i][1] * fast_exp2(b.y - ref_q[1]), hi, lo);
+          const Pair bq = padd(b, Pair{-ref_q.x, -ref_q.y}), q = pmul(qv[i], Pair{fast_exp2(bq.x), fast_exp2(bq.y)});
+          split2(q.x, q.y, hi, lo);
           *reinterpret_cast<uint32_t*>(sm + T_Q + at) = hi;
           *reinterpret_cast<uint32_t*>(sm + T_Q + T_SPLIT + at) = lo;
         }
       }
       fence_proxy_async_smem();
       tc_fence_before();
-      mbar_arrive_warp(b_qk);
-      mbar_arrive_warp(b_free);
-      lc_meet();                                          // factors of the state
-      // ---- state: operand of the product with Q, and the sum that K^T V is added to
-      {
+      if (OUT) {
+        mbar_arrive_warp(b_qk);
+        mbar_arrive_warp(b_free);
+        lc_meet();                                        // factors of the state
+      } else {
+        mbar_arrive_warp(b_free);
+      }
+      if (OUT) {
+        // ---- state: operand of the product with Q, and the sum that K^T V is added to
         uint32_t r[32], hi[16], lo[16];
         __syncwarp();
         tmem_ld32(tmem + TM_S + lanes + cg * 32, r);
@@ -349,24 +347,20 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
 #pragma unroll
         for (int j = 0; j < 32; j += 4) {
           const float4 w0 = *reinterpret_cast<const float4*>(f0 + cg * 32 + j), wk = *reinterpret_cast<const float4*>(fk + cg * 32 + j);
-          const float x0 = __uint_as_float(r[j]) * w0.x, x1 = __uint_as_float(r[j + 1]) * w0.y, x2 = __uint_as_float(r[j + 2]) * w0.z,
-                      x3 = __uint_as_float(r[j + 3]) * w0.w;
-          const float y0 = x0 * wk.x, y1 = x1 * wk.y, y2 = x2 * wk.z, y3 = x3 * wk.w;
-          if (OUT) {
-            split2(far ? x0 : y0, far ? x1 : y1, hi[j / 2], lo[j / 2]);
-            split2(far ? x2 : y2, far ? x3 : y3, hi[j / 2 + 1], lo[j / 2 + 1]);
-          }
-          r[j] = __float_as_uint(y0);
-          r[j + 1] = __float_as_uint(y1);
-          r[j + 2] = __float_as_uint(y2);
-          r[j + 3] = __float_as_uint(y3);
+          const Pair x0 = pmul(Pair{__uint_as_float(r[j]), __uint_as_float(r[j + 1])}, Pair{w0.x, w0.y});
+          const Pair x1 = pmul(Pair{__uint_as_float(r[j + 2]), __uint_as_float(r[j + 3])}, Pair{w0.z, w0.w});
+          const Pair y0 = pmul(x0, Pair{wk.x, wk.y}), y1 = pmul(x1, Pair{wk.z, wk.w});
+          split2(far ? x0.x : y0.x, far ? x0.y : y0.y, hi[j / 2], lo[j / 2]);
+          split2(far ? x1.x : y1.x, far ? x1.y : y1.y, hi[j / 2 + 1], lo[j / 2 + 1]);
+          r[j] = __float_as_uint(y0.x);
+          r[j + 1] = __float_as_uint(y0.y);
+          r[j + 2] = __float_as_uint(y1.x);
+          r[j + 3] = __float_as_uint(y1.y);
         }
         __syncwarp();
         tmem_st32(tmem + TM_S + lanes + cg * 32, r);
-        if (OUT) {
-          tmem_st16(tmem + TM_SH + lanes + cg * 16, hi);
-          tmem_st16(tmem + TM_SL + lanes + cg * 16, lo);
-        }
+        tmem_st16(tmem + TM_SH + lanes + cg * 16, hi);
+        tmem_st16(tmem + TM_SL + lanes + cg * 16, lo);
         tmem_st_wait();
       }
       if (OUT && !far) {
@@ -396,7 +390,7 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
       fence_proxy_async_smem();
       tc_fence_before();
       mbar_arrive_warp(b_sa);
-      if (n + 1 < n_chunks) gates(n + 1);                 // while the tensor core works
+      if (n + 1 < n_chunks) gates(n + 1, chunk_of(n + 1));                 // while the tensor core works
       if (OUT) {
         // ---- result: lane = element of v, this warp's 16 tokens; norm over the head, gate.  Rows go through the tile of Q
         // (its products are done) to leave in 16-byte pieces.
@@ -431,7 +425,7 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
         for (int i = 0; i < 2; ++i) {
           const int t = o_row + 8 * i;
           if (!o_mine || t >= left) continue;
-          const float scale = 1.0f / sqrtf((red[t] + red[LC + t] + red[2 * LC + t] + red[3 * LC + t]) / V + a.eps);
+          const float scale = rsqrtf(fmaf(red[t] + red[LC + t] + red[2 * LC + t] + red[3 * LC + t], inv_v, a.eps));
           const float4 x0 = *reinterpret_cast<const float4*>(rows + t * 128 + o_col), x1 = *reinterpret_cast<const float4*>(rows + t * 128 + o_col + 4);
           const float4 w0 = *reinterpret_cast<const float4*>(a.w + o_col), w1 = *reinterpret_cast<const float4*>(a.w + o_col + 4);
           float x[8] = {x0.x * scale * w0.x, x0.y * scale * w0.y, x0.z * scale * w0.z, x0.w * scale * w0.w,
@@ -454,7 +448,10 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
     if (n_chunks > 0) ok &= mbar_wait(bar_s, (n_chunks - 1) & 1, dead, c.status, 803);
     tc_fence_after();
     lc_meet();
-    if (tg == 0) { f0[ch] = exp2f(pend[0]); f0[ch + 1] = exp2f(pend[1]); }
+    if (tg == 0) {
+      f0[ch] = OUT ? exp2f(pend.x) : 1.0f;
+      f0[ch + 1] = OUT ? exp2f(pend.y) : 1.0f;
+    }
     lc_meet();
     if (ok && (!OUT || last)) {
       uint32_t r[32];
@@ -468,8 +465,8 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
         if (lrow < V && cg * 32 + j < D) dst[(long long)(cg * 32 + j) * V + lrow] = __uint_as_float(r[j]) * f0[cg * 32 + j];
       if (!OUT && tg == 0 && mine) {
         float* total = c.total + ((long long)blockIdx.y * a.heads + h) * D + ch;
-        total[0] = tot[0];
-        total[1] = tot[1];
+        total[0] = tot.x;
+        total[1] = tot.y;
       }
     }
   }
