@@ -7,8 +7,9 @@
 // two bf16 numbers, so the sums see 16 bits of each factor; the two parts of Q, K and A are stacked in one tile, which
 // makes the partial products one wider instruction:
 //     [Qh; Ql] [Kh; Kl]^T  -> A in four quarters        Sh [Qh; Ql]^T, Sl Qh^T, V^T [Ah; Al]^T  -> O^T in two halves
-// Where a decay is so strong that the exponents could leave fp32's range, A is formed term by term with
-// b_t - b_s <= 0, and Q and K take the chunk's ends as their references.
+// Where a state row's decay is so strong that its exponents could leave fp32's range, the row's part of A is formed term by
+// term with b_t - b_s <= 0, and its columns of Q and K take the chunk's ends as their references (what the product
+// makes of them is below 2^-100 of the truth).
 //
 // One CTA walks the chunks of one (stretch of a run, head).  A long run is cut into stretches that run side by side: a
 // first pass sums up what each stretch adds to the state, a second one turns that into the stretches' first states.
@@ -25,7 +26,8 @@ constexpr int LC = 64, LC_THREADS = 512;                  // tokens of a chunk; 
 constexpr float LC_LIMIT = 100.0f;                        // largest exponent (base 2) of a factor
 // shared memory (bytes): operand tiles of 128-byte rows in blocks of 64 columns, then rows as they come from memory
 constexpr uint32_t T_Q = 0, T_K = 32768, T_V = 65536, T_A = 81920, T_A2 = 98304, R_Z = 106496, R_W = R_Z + 32768, R_X = R_W + 16384, LC_MISC = R_X + 16384;
-constexpr uint32_t LC_SMEM = LC_MISC + (8 * 128 + 5 * 128 + 4 * LC) * 4 + 128 + 1024;
+constexpr int FAR_N = 24;                                 // strongly decaying state rows handled at a time
+constexpr uint32_t LC_SMEM = LC_MISC + (8 * 128 + 3 * 128 + 4 * LC + LC * LC + FAR_N * 3 * LC) * 4 + 128 + 1024;
 constexpr uint32_t T_SPLIT = 8192;                        // high part -> low part of Q, K and A: 64 rows further
 // TMEM columns: state, its two parts, O in two halves, A in four quarters
 constexpr uint32_t TM_S = 0, TM_SH = 128, TM_SL = 192, TM_O = 256, TM_A = 384;
@@ -89,14 +91,17 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
   uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lc_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sb = smem_u32(sm);
   float* part = reinterpret_cast<float*>(sm + LC_MISC);   // [8][128] decay of eight tokens
-  float* f0 = part + 8 * 128;                             // [128] factors of the state: pending, of K's reference
+  float* f0 = part + 8 * 128;                             // [128] factors of the state: pending, of K's and Q's references
   float* fk = f0 + 128;
-  float* red = fk + 128;                                  // [4][64]
-  uint32_t* bars = reinterpret_cast<uint32_t*>(red + 4 * LC);
+  float* fq = fk + 128;
+  float* red = fq + 128;                                  // [4][64]
+  float* far_a = red + 4 * LC;                            // [64][64] what strongly decaying rows give to A
+  float* far_rows = far_a + LC * LC;                      // [FAR_N][q, k, b][64]
+  uint32_t* bars = reinterpret_cast<uint32_t*>(far_rows + FAR_N * 3 * LC);
   const uint32_t b_qk = smem_u32(bars), b_sa = b_qk + 8, bar_a = b_qk + 16, bar_o = b_qk + 24, bar_s = b_qk + 32, b_raw = b_qk + 40, b_free = b_qk + 48, b_v = b_qk + 56;
   volatile uint32_t* tmem_slot = bars + 16;
   volatile int* dead = reinterpret_cast<volatile int*>(bars + 17);
-  volatile int* far_flag = reinterpret_cast<volatile int*>(bars + 18);
+  uint32_t* far_mask = bars + 18;                         // [4]
 
   const int* item = c.items + 4 * blockIdx.y;
   const int row0 = item[0], count = item[1], last = item[3], h = blockIdx.x;
@@ -158,15 +163,10 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
       if (OUT) {
         if (!__all_sync(0xffffffffu, mbar_wait(b_qk, n & 1, dead, c.status, 810))) break;
         tc_fence_after();
-        if (*far_flag) {
-          if (mine) mbar_arrive(bar_a);
-          __syncwarp();
-        } else {
 #pragma unroll
-          for (int kk = 0; kk < 8; ++kk)
-            if (kk < ksteps) umma_f16_lane(mine, tm + TM_A, k_major(dq, kk), k_major(dk, kk), id_kk, kk != 0);
-          umma_commit_lane(mine, bar_a);
-        }
+        for (int kk = 0; kk < 8; ++kk)
+          if (kk < ksteps) umma_f16_lane(mine, tm + TM_A, k_major(dq, kk), k_major(dk, kk), id_kk, kk != 0);
+        umma_commit_lane(mine, bar_a);
       }
       if (!__all_sync(0xffffffffu, mbar_wait(b_v, n & 1, dead, c.status, 812) && mbar_wait(b_sa, n & 1, dead, c.status, 811))) break;
       tc_fence_after();
@@ -266,50 +266,59 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
       auto sum_at = [&](int i) {                          // decay up to and with this thread's token i
         return mine ? padd(*reinterpret_cast<const Pair*>(sm + R_Z + ((tg * 8 + i) * D + ch) * 4), before) : pall(0.0f);
       };
-      bool far = false;
-      if (OUT) far = lc_any(fmaxf(-mid.x, -mid.y) > LC_LIMIT || fmaxf(mid.x - end.x, mid.y - end.y) > LC_LIMIT);
+      const bool far_x = OUT && (-mid.x > LC_LIMIT || mid.x - end.x > LC_LIMIT), far_y = OUT && (-mid.y > LC_LIMIT || mid.y - end.y > LC_LIMIT);
+      const bool far = OUT && lc_any(far_x || far_y);
       if (far) {
-        // A term by term: row tid / 8, columns 8 (tid % 8) ..; scratch space: the tiles of Q and K, and b in its own rows
-        float* fx = reinterpret_cast<float*>(sm + T_Q);
-        float* fy = reinterpret_cast<float*>(sm + T_K);
-        float* fb = reinterpret_cast<float*>(sm + R_Z);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const int at = (tg * 8 + i) * 128 + ch;
-          *reinterpret_cast<Pair*>(fx + at) = qv[i];
-          *reinterpret_cast<Pair*>(fy + at) = kv[i];
-          if (mine) *reinterpret_cast<Pair*>(fb + (tg * 8 + i) * D + ch) = sum_at(i);
+        // number the rows, bring theirs together, and work out their part of A: row tid / 8, columns 8 (tid % 8) ..
+        if (warp < 2) {
+          const uint32_t mx = __ballot_sync(0xffffffffu, far_x), my = __ballot_sync(0xffffffffu, far_y);
+          if (lane == 0) { far_mask[2 * warp] = mx; far_mask[2 * warp + 1] = my; }
         }
-        before = pall(0.0f);                              // b's rows are complete now
         lc_meet();
+        const int w = (tid >> 5) & 1, below0 = w ? __popc(far_mask[0]) + __popc(far_mask[1]) : 0;
+        const uint32_t below = (1u << lane) - 1u;
+        const int ix = below0 + __popc(far_mask[2 * w] & below) + __popc(far_mask[2 * w + 1] & below), iy = ix + far_x;
+        const int n_far = __popc(far_mask[0]) + __popc(far_mask[1]) + __popc(far_mask[2]) + __popc(far_mask[3]);
         const int t = tid >> 3, s0 = (tid & 7) * 8;
-        uint32_t hi[4], lo[4];
+        float acc[8];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          float x[2] = {0.0f, 0.0f};
+        for (int j = 0; j < 8; ++j) acc[j] = 0.0f;
+        for (int g0 = 0; g0 < n_far; g0 += FAR_N) {
+          const bool put_x = far_x && ix >= g0 && ix < g0 + FAR_N, put_y = far_y && iy >= g0 && iy < g0 + FAR_N;
 #pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            const int s = s0 + 2 * j + i;
-            if (s <= t)
-#pragma unroll 1
-              for (int e = 0; e < D; ++e) x[i] = fmaf(fx[t * 128 + e] * fy[s * 128 + e], exp2f(fb[t * D + e] - fb[s * D + e]), x[i]);
+          for (int i = 0; i < 8; ++i) {
+            const Pair b = sum_at(i);
+            float* px = far_rows + (ix - g0) * 3 * LC + tg * 8 + i;
+            float* py = far_rows + (iy - g0) * 3 * LC + tg * 8 + i;
+            if (put_x) { px[0] = qv[i].x; px[LC] = kv[i].x; px[2 * LC] = b.x; }
+            if (put_y) { py[0] = qv[i].y; py[LC] = kv[i].y; py[2 * LC] = b.y; }
           }
-          split2(x[0], x[1], hi[j], lo[j]);
+          lc_meet();
+          if (s0 <= t)
+            for (int r = 0; r < min(FAR_N, n_far - g0); ++r) {
+              const float* row = far_rows + r * 3 * LC;
+              const float q = row[t], b = row[2 * LC + t];
+#pragma unroll
+              for (int j = 0; j < 8; ++j)
+                if (s0 + j <= t) acc[j] = fmaf(q * row[LC + s0 + j], fast_exp2(b - row[2 * LC + s0 + j]), acc[j]);
+            }
+          lc_meet();
         }
-        lc_meet();
-        const uint32_t at = sw128_offset(t, s0 >> 3);
-        *reinterpret_cast<uint4*>(sm + T_A + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *reinterpret_cast<uint4*>(sm + T_A + T_SPLIT + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-        *reinterpret_cast<uint4*>(sm + T_A2 + at) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<float4*>(far_a + t * LC + s0) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        *reinterpret_cast<float4*>(far_a + t * LC + s0 + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
       }
       // K's factors refer to the chunk's middle or end; the summing pass comes from the end and adds what follows
-      const Pair ref_q = far ? pall(0.0f) : mid, ref_k = OUT ? (far ? end : mid) : padd(end, tot);
+      const Pair ref_q = {far_x ? 0.0f : mid.x, far_y ? 0.0f : mid.y};
+      const Pair ref_k = OUT ? Pair{far_x ? end.x : mid.x, far_y ? end.y : mid.y} : padd(end, tot);
       if (OUT && tg == 0) {
         f0[ch] = exp2f(pend.x);
         f0[ch + 1] = exp2f(pend.y);
-        fk[ch] = exp2f(ref_k.x);                          // Q's reference is the same, or 0
+        fk[ch] = exp2f(ref_k.x);
         fk[ch + 1] = exp2f(ref_k.y);
-        if (tid == 0) *far_flag = far;
+        if (far) {                                        // otherwise Q has K's references
+          fq[ch] = exp2f(ref_q.x);
+          fq[ch + 1] = exp2f(ref_q.y);
+        }
       }
       pend = padd(end, Pair{-ref_k.x, -ref_k.y});
       tot = padd(tot, end);
@@ -350,8 +359,14 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
           const Pair x0 = pmul(Pair{__uint_as_float(r[j]), __uint_as_float(r[j + 1])}, Pair{w0.x, w0.y});
           const Pair x1 = pmul(Pair{__uint_as_float(r[j + 2]), __uint_as_float(r[j + 3])}, Pair{w0.z, w0.w});
           const Pair y0 = pmul(x0, Pair{wk.x, wk.y}), y1 = pmul(x1, Pair{wk.z, wk.w});
-          split2(far ? x0.x : y0.x, far ? x0.y : y0.y, hi[j / 2], lo[j / 2]);
-          split2(far ? x1.x : y1.x, far ? x1.y : y1.y, hi[j / 2 + 1], lo[j / 2 + 1]);
+          Pair z0 = y0, z1 = y1;
+          if (far) {
+            const float4 wq = *reinterpret_cast<const float4*>(fq + cg * 32 + j);
+            z0 = pmul(x0, Pair{wq.x, wq.y});
+            z1 = pmul(x1, Pair{wq.z, wq.w});
+          }
+          split2(z0.x, z0.y, hi[j / 2], lo[j / 2]);
+          split2(z1.x, z1.y, hi[j / 2 + 1], lo[j / 2 + 1]);
           r[j] = __float_as_uint(y0.x);
           r[j + 1] = __float_as_uint(y0.y);
           r[j + 2] = __float_as_uint(y1.x);
@@ -363,7 +378,7 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
         tmem_st16(tmem + TM_SL + lanes + cg * 16, lo);
         tmem_st_wait();
       }
-      if (OUT && !far) {
+      if (OUT) {
         // ---- A, lower triangle: the quarters of Qh (lanes 0 .. 63) as two bf16 parts, those of Ql as one
         ok &= mbar_wait(bar_a, n & 1, dead, c.status, 800);
         tc_fence_after();
@@ -379,8 +394,9 @@ linear_chunks_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_cons
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int i = j + 2 * e, s = cg * 16 + i;
-            split2(s <= t ? __uint_as_float(r[i]) + __uint_as_float(r2[i]) : 0.0f,
-                   s + 1 <= t ? __uint_as_float(r[i + 1]) + __uint_as_float(r2[i + 1]) : 0.0f, hi[e], lo[e]);
+            Pair x = {s <= t ? __uint_as_float(r[i]) + __uint_as_float(r2[i]) : 0.0f, s + 1 <= t ? __uint_as_float(r[i + 1]) + __uint_as_float(r2[i + 1]) : 0.0f};
+            if (far && quad < 2) x = padd(x, *reinterpret_cast<const Pair*>(far_a + t * LC + s));
+            split2(x.x, x.y, hi[e], lo[e]);
           }
           const uint32_t at = sw128_offset(t, (cg * 16 + j) >> 3);
           *reinterpret_cast<uint4*>(sm + (quad < 2 ? T_A : T_A2) + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
