@@ -172,7 +172,7 @@ class HybridCache(PagedCache):
             n = min(self.ROWS, N - i)
             if splits <= 0:
                 ctas = n * s.heads * (1 if group <= 2 else (group + 3) // 4)
-                splits = max(1, min(32, 592 // ctas, (longest + 63) // 64))
+                splits = max(1, min(32, 1536 // ctas, (longest + 63) // 64))
             need = L.cgk_kv_rows_scratch_floats(n, H, s.vdim, splits)
             scratch = torch.empty(need, dtype=torch.float32, device=q.device) if need else None
             a = self._args(layer, slot[i:], pos[i:])

@@ -212,12 +212,40 @@ __device__ __forceinline__ void finish_pair(const RowsDev& a, long long t, int h
 }
 
 // One CTA = (key range, kv head with up to R of its query heads, query token).  LPK lanes share a key, EPL elements each;
-// the 32 / LPK key groups of a warp and the four warps keep running maxima of their own and are merged at the end.
+// a warp takes U keys per group of lanes at a time, the next ones on their way while it works.  The U * R scores are summed
+// over the lanes so that every lane ends with its share of them (and one exponential per score is computed); maxima are
+// the warp's, and stay until a score passes one by more than 2^8.  The four warps are merged at the end.
 constexpr int KR_WARPS = 4;
+template <int N, int LPK>
+struct Shares {                                         // N sums over LPK lanes: C per lane, or DUP lanes with the same one
+  static constexpr int C = N > LPK ? N / LPK : 1, DUP = N < LPK ? LPK / N : 1;
+  static __device__ __forceinline__ int index(int sub, int c) { return DUP > 1 ? sub / DUP : sub * C + c; }
+  static __device__ __forceinline__ int lane_of(int i) { return DUP > 1 ? i * DUP : i / C; }
+  template <int M, int OFF>
+  static __device__ __forceinline__ void step(float (&v)[N], int sub) {
+    if constexpr (OFF >= 1) {
+      if constexpr (M > 1) {
+        const bool upper = (sub & OFF) != 0;
+#pragma unroll
+        for (int i = 0; i < M / 2; ++i) {
+          const float send = upper ? v[i] : v[i + M / 2];
+          v[i] = (upper ? v[i + M / 2] : v[i]) + __shfl_xor_sync(0xffffffffu, send, OFF);
+        }
+        step<M / 2, OFF / 2>(v, sub);
+      } else {
+        v[0] += __shfl_xor_sync(0xffffffffu, v[0], OFF);
+        step<1, OFF / 2>(v, sub);
+      }
+    }
+  }
+  static __device__ __forceinline__ void sum(float (&v)[N], int sub) { step<N, LPK / 2>(v, sub); }
+};
+
 template <typename T, int LPK, int EPL, int R>
-__global__ void __launch_bounds__(KR_WARPS * 32)
+__global__ void __launch_bounds__(KR_WARPS * 32, sizeof(T) == 2 && EPL == 8 ? 3 : 1)
 kv_rows_kernel(const RowsDev a) {
-  constexpr int KPW = 32 / LPK, W = LPK * EPL, KR_U = EPL == 8 ? 4 : 1;
+  constexpr int KPW = 32 / LPK, W = LPK * EPL, U = EPL == 8 ? 4 : 1, N = U * R;
+  typedef Shares<N, LPK> Sh;
   __shared__ float sh[KR_WARPS][R][W];
   __shared__ float stat[KR_WARPS][R][2];
   const KvRowsDev& c = a.c;
@@ -227,18 +255,19 @@ kv_rows_kernel(const RowsDev a) {
   const int group = a.heads / c.kv_heads, h0 = g * group + hg * R, nh = min(R, group - hg * R);
   const int p = (int)CGK_IDX(c.pos[t], (long long)c.max_pages * c.page_size);
   const int lo = a.block > 0 ? p / a.block * a.block : 0, n = p + 1 - lo;
-  constexpr int STEP = KR_WARPS * KPW * KR_U;
+  constexpr int STEP = KR_WARPS * KPW * U;
   const int per = ((n + a.splits - 1) / a.splits + STEP - 1) / STEP * STEP;
   const int k_begin = lo + split * per, k_end = min(p + 1, k_begin + per);
   const int* row = c.page_table + CGK_IDX(c.slot[t], c.slots) * c.max_pages;
   const T* kp = reinterpret_cast<const T*>(c.k_pages);
   const T* vp = reinterpret_cast<const T*>(c.v_pages);
 
-  float q[R][EPL], acc[R][EPL], m[R], l[R];
+  float q[R][EPL], acc[R][EPL], m[R], l[Sh::C], mo[Sh::C];
+#pragma unroll
+  for (int i = 0; i < Sh::C; ++i) { l[i] = 0.0f; mo[i] = -INFINITY; }
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     m[r] = -INFINITY;
-    l[r] = 0.0f;
 #pragma unroll
     for (int e = 0; e < EPL; ++e) { q[r][e] = 0.0f; acc[r][e] = 0.0f; }
     if (r < nh) {
@@ -249,63 +278,75 @@ kv_rows_kernel(const RowsDev a) {
       for (int e = 0; e < EPL; ++e) q[r][e] *= a.scale_log2;
     }
   }
-  for (int k0 = k_begin + warp * KPW * KR_U; k0 < k_end; k0 += STEP) {
-    float s[KR_U][R];
-    RawRow<T, EPL> kk[KR_U], vv[KR_U];
+  RawRow<T, EPL> kk[U], vv[U];
+  auto load = [&](int k0) {
 #pragma unroll
-    for (int u = 0; u < KR_U; ++u) {
+    for (int u = 0; u < U; ++u) {
       const int key = min(k0 + u * KPW + kg, k_end - 1);
       const long long at = c.row_of(CGK_IDX(row[c.page_of(key)], c.n_pages), g, key);
       kk[u].load(kp + at * c.ld_k, e0, c.ld_k);
       vv[u].load(vp + at * c.ld_v, e0, c.ld_v);
     }
+  };
+  int k0 = k_begin + warp * KPW * U;
+  if (k0 < k_end) load(k0);
+  for (; k0 < k_end; k0 += STEP) {
+    float s[N];
 #pragma unroll
-    for (int u = 0; u < KR_U; ++u) {
+    for (int u = 0; u < U; ++u) {
       float x[EPL];
       kk[u].get(x);
 #pragma unroll
       for (int r = 0; r < R; ++r) {
-        float d = 0.0f;
+        float d0 = 0.0f, d1 = 0.0f;
 #pragma unroll
-        for (int e = 0; e < EPL; ++e) d = fmaf(q[r][e], x[e], d);
-        s[u][r] = d;
+        for (int e = 0; e < EPL; e += 2) ffma2(d0, d1, q[r][e], q[r][e + 1], x[e], x[e + 1], d0, d1);
+        s[u * R + r] = d0 + d1;
       }
     }
+    RawRow<T, EPL> v0[U];
 #pragma unroll
-    for (int u = 0; u < KR_U; ++u) {
-      const bool vis = k0 + u * KPW + kg < k_end;
+    for (int u = 0; u < U; ++u) v0[u] = vv[u];
+    const int k1 = k0;
+    if (k0 + STEP < k_end) load(k0 + STEP);
+    Sh::sum(s, sub);
+    bool grown = false;
 #pragma unroll
-      for (int r = 0; r < R; ++r) {
-#pragma unroll
-        for (int o = LPK / 2; o > 0; o >>= 1) s[u][r] += __shfl_xor_sync(0xffffffffu, s[u][r], o);
-        if (!vis) s[u][r] = -INFINITY;
-      }
+    for (int i = 0; i < Sh::C; ++i) {
+      if (k1 + Sh::index(sub, i) / R * KPW + kg >= k_end) s[i] = -INFINITY;
+      grown |= s[i] > mo[i] + 8.0f;
     }
-    if (k0 + kg < k_end) {                              // this key group has a key (its first one) in the range
+    if (__any_sync(0xffffffffu, grown)) {
 #pragma unroll
       for (int r = 0; r < R; ++r) {
-        float mn = m[r];
+        float x = -INFINITY;
 #pragma unroll
-        for (int u = 0; u < KR_U; ++u) mn = fmaxf(mn, s[u][r]);
-        const float corr = exp2f(m[r] - mn);
-        l[r] *= corr;
-        m[r] = mn;
+        for (int i = 0; i < Sh::C; ++i) x = Sh::index(sub, i) % R == r ? fmaxf(x, s[i]) : x;
+        x = fmaxf(warp_max(x), m[r]);
+        const float corr = x > -INFINITY ? exp2f(m[r] - x) : 1.0f;
+        m[r] = x;
 #pragma unroll
         for (int e = 0; e < EPL; ++e) acc[r][e] *= corr;
 #pragma unroll
-        for (int u = 0; u < KR_U; ++u) {
-          s[u][r] = exp2f(s[u][r] - mn);
-          l[r] += s[u][r];
-        }
+        for (int i = 0; i < Sh::C; ++i)
+          if (Sh::index(sub, i) % R == r) { l[i] *= corr; mo[i] = x; }
       }
+    }
+    float w[Sh::C];
 #pragma unroll
-      for (int u = 0; u < KR_U; ++u) {
-        float x[EPL];
-        vv[u].get(x);
+    for (int i = 0; i < Sh::C; ++i) {
+      w[i] = sizeof(T) == 2 ? fast_exp2(s[i] - mo[i]) : exp2f(s[i] - mo[i]);
+      l[i] += w[i];
+    }
 #pragma unroll
-        for (int r = 0; r < R; ++r)
+    for (int u = 0; u < U; ++u) {
+      float x[EPL];
+      v0[u].get(x);
 #pragma unroll
-          for (int e = 0; e < EPL; ++e) acc[r][e] = fmaf(s[u][r], x[e], acc[r][e]);
+      for (int r = 0; r < R; ++r) {
+        const float pw = __shfl_sync(0xffffffffu, w[(u * R + r) % Sh::C], kg * LPK + Sh::lane_of(u * R + r));
+#pragma unroll
+        for (int e = 0; e < EPL; e += 2) ffma2(acc[r][e], acc[r][e + 1], pw, pw, x[e], x[e + 1], acc[r][e], acc[r][e + 1]);
       }
     }
   }
@@ -313,22 +354,19 @@ kv_rows_kernel(const RowsDev a) {
 #pragma unroll
   for (int r = 0; r < R; ++r) {
 #pragma unroll
-    for (int o = LPK; o < 32; o <<= 1) {
-      const float mo = __shfl_xor_sync(0xffffffffu, m[r], o), lo2 = __shfl_xor_sync(0xffffffffu, l[r], o), mn = fmaxf(m[r], mo);
-      const float f = m[r] > -INFINITY ? exp2f(m[r] - mn) : 0.0f, fo = mo > -INFINITY ? exp2f(mo - mn) : 0.0f;
-      l[r] = l[r] * f + lo2 * fo;
-      m[r] = mn;
+    for (int e = 0; e < EPL; ++e)
 #pragma unroll
-      for (int e = 0; e < EPL; ++e) {
-        const float x = __shfl_xor_sync(0xffffffffu, acc[r][e], o);
-        acc[r][e] = acc[r][e] * f + x * fo;
-      }
-    }
+      for (int o = LPK; o < 32; o <<= 1) acc[r][e] += __shfl_xor_sync(0xffffffffu, acc[r][e], o);
+    float lr = 0.0f;
+#pragma unroll
+    for (int i = 0; i < Sh::C; ++i)
+      if (Sh::index(sub, i) % R == r && sub % Sh::DUP == 0) lr += l[i];
+    lr = warp_sum(lr);
     if (kg == 0) {
 #pragma unroll
       for (int e = 0; e < EPL; ++e) sh[warp][r][e0 + e] = acc[r][e];
     }
-    if (lane == 0) { stat[warp][r][0] = m[r]; stat[warp][r][1] = l[r]; }
+    if (lane == 0) { stat[warp][r][0] = m[r]; stat[warp][r][1] = lr; }
   }
   __syncthreads();
   const int pairs = (c.vdim + 1) / 2;
