@@ -233,10 +233,12 @@ static int launch_grouped(const cgk_gemm_args& a, const GemmDev& g0, int sms, cu
   g.tiles_m = (a.M + BM - 1) / BM;
   g.tiles_n = (a.N + BN - 1) / BN;
   CUtensorMap tmA, tmB, tmC, tmAux, tmIn;
-  int rc = make_gemm_tmaps(a, BN, &tmA, &tmB);
-  if (rc) return rc;
+  // A and the output are one matrix each: a map of A with B's batch size would reach far beyond its memory
   cgk_gemm_args one = a;
   one.batch = 1;
+  CUtensorMap first_b;
+  int rc = make_gemm_tmaps(one, BN, &tmA, &first_b);
+  if (rc || (rc = make_gemm_tmaps(a, BN, &first_b, &tmB))) return rc;
   int out_ok = 0, in_kind = 0;
   if ((rc = make_gemm_out_tmaps(one, &tmC, &tmAux, &tmIn, &out_ok, &in_kind))) return rc;
   g.tma_store = out_ok ? 1 : 0;
@@ -257,7 +259,7 @@ CGK_API int cgk_gemm_grouped_bf16(const cgk_gemm_args* pa, const int* tile_group
   CGK_REQUIRE(!a.a_mn && !a.b_mn && !a.accumulate && !a.bias && !a.act && !a.residual && !a.aux_out && !a.aux_in && !a.rope_cos && a.alpha == 1.0f,
               "cgk_gemm_grouped_bf16: plain K-major products only");
   if (a.M == 0 || a.N == 0) return 0;
-  a.strideA = (int64_t)a.M * a.lda;                    // A is one matrix: only its first batch entry is addressed
+  a.strideA = (int64_t)a.M * a.lda;
   CGK_REQUIRE(gemm_tma_ok(a) && a.M % BM == 0, "cgk_gemm_grouped_bf16: operands must satisfy the TMA alignment rules, rows whole tiles");
   int dev = 0;
   CGK_CUDA_CHECK(cudaGetDevice(&dev));
