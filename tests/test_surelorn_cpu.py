@@ -291,7 +291,8 @@ def test_the_serving_subset_of_the_kernels_has_what_the_engine_calls(tmp_path):
     so = build.build_serving_kernels(out=tmp_path / "serve.so")
     lib = ctypes.CDLL(str(so))
     named = set()
-    for f in ("ops/stream.py", "ops/moe.py", "ops/linear.py", "ops/gemm.py", "serve/kv_cache.py", "serve/sampling.py"):
+    for f in ("ops/stream.py", "ops/moe.py", "ops/linear.py", "ops/gemm.py", "ops/recurrence.py", "ops/rotary.py", "serve/kv_cache.py",
+              "serve/hybrid_cache.py", "serve/sampling.py"):
         named |= set(re.findall(r"\.(cgk_\w+)\(", (root / "cogito_b200" / f).read_text()))
     assert len(named) > 15 and not [n for n in named if not hasattr(lib, n)]
     # the bindings accept a library without the training kernels
